@@ -182,6 +182,44 @@ def _cmd_bench(args, rest: Sequence[str]) -> int:
     return subprocess.call([sys.executable, os.path.join(root, "bench.py"), *rest])
 
 
+def _cmd_generate(args) -> int:
+    """Token ids in, token ids out: ``Model.sample_decode`` on a checkpoint folder (the decode engine
+    behind it on a GPU)."""
+    import torch  # pylint: disable=import-outside-toplevel
+
+    from axlearn_b200.common import logit_modifiers, prng  # pylint: disable=import-outside-toplevel
+    from axlearn_b200.common.module import functional  # pylint: disable=import-outside-toplevel
+    from axlearn_b200.inference.model_loader import load_model  # pylint: disable=import-outside-toplevel
+
+    dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}[args.dtype]
+    prompts = [[int(t) for t in p.replace(",", " ").split()] for p in args.prompt]
+    loaded = load_model(args.model, dtype=dtype, device=args.device)
+    cfg = loaded.decoder.config
+    vocab, pad = cfg.vocab_size, cfg.pad_token_id
+    if any(not p or min(p) < 0 or max(p) >= vocab or p[-1] == pad for p in prompts):
+        raise SystemExit(f"prompts are token ids in [0, {vocab}) and do not end in the padding id {pad}")
+    longest = max(len(p) for p in prompts)
+    prefix = torch.full((len(prompts), longest), pad, dtype=torch.int64, device=args.device)
+    for row, p in enumerate(prompts):
+        prefix[row, :len(p)] = torch.tensor(p)
+    modifiers = []
+    if args.temperature == 0:
+        modifiers.append(logit_modifiers.top_k_logits(1))
+    elif args.top_k:
+        modifiers.append(logit_modifiers.top_k_logits(args.top_k))
+    with torch.no_grad():
+        out, _ = functional(
+            loaded.model, prng.PRNGKey(args.seed), loaded.parameters,
+            dict(input_batch={"prefix": prefix}, max_sequence_length=longest + args.max_new_tokens + 1,
+                 temperature=args.temperature or 1.0, logits_modifier=modifiers[0] if modifiers else None),
+            method="sample_decode", is_training=False)
+    for row, p in enumerate(prompts):
+        # Sequences leave out the first (conditioning) token of the prompt.
+        ids = out.sequences[row, 0, len(p) - 1:len(p) - 1 + args.max_new_tokens].tolist()
+        print(json.dumps({"prompt": p, "tokens": ids}))
+    return 0
+
+
 def build_parser() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser(prog="axlearn_b200")
     groups = ap.add_subparsers(dest="group", required=True)
@@ -189,6 +227,18 @@ def build_parser() -> argparse.ArgumentParser:
     train = groups.add_parser("train", help="run a trainer config; unknown flags go to launch_trainer_main")
     train.add_argument("--gpus", type=int, default=1)
     groups.add_parser("bench", help="run bench.py; flags are passed through")
+
+    gen = groups.add_parser("generate", help="decode token ids from a checkpoint folder")
+    gen.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
+    gen.add_argument("--prompt", action="append", required=True, help="token ids, e.g. '12 7 9'; repeat for a batch")
+    gen.add_argument("--max_new_tokens", type=int, default=16)
+    gen.add_argument("--temperature", type=float, default=0.0, help="0 = greedy")
+    gen.add_argument("--top_k", type=int, default=0)
+    gen.add_argument("--seed", type=int, default=0)
+    gen.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    gen.add_argument("--device", default="cuda")
+    trace = groups.add_parser("trace", help="replay given token ids step by step; flags go to inference/trace.py")
+    trace.add_argument("rest", nargs=argparse.REMAINDER)
 
     bastion = groups.add_parser("bastion")
     bastion.add_argument("action", choices=["start", "submit", "cancel", "list", "state"])
@@ -251,6 +301,10 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
         return _cmd_bench(args, rest)
     if args.group == "gcp":
         return _cmd_gcp(args, rest)
+    if args.group == "trace":
+        from axlearn_b200.inference import trace  # pylint: disable=import-outside-toplevel
+
+        return trace.main(list(args.rest) + list(rest))
     if rest:
         raise SystemExit(f"unknown arguments: {rest}")
     if args.group == "bastion":
@@ -261,4 +315,6 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
         if args.action == "submit" and not args.command:
             raise SystemExit("bastion submit needs --command")
         return _cmd_bastion(args)
+    if args.group == "generate":
+        return _cmd_generate(args)
     return _cmd_bundle(args)

@@ -152,7 +152,8 @@ class Decoder(BaseLayer):
     # ------------------------------------------------------------------ core
     def _forward_for_mode(self, *, mode: ForwardMode, input_batch: dict, cached_states=None,
                           cross_attention_data=None, cross_attention_logit_biases=None,
-                          self_attention_logit_biases=None, page_pool=None, max_len=None, **kwargs):
+                          self_attention_logit_biases=None, page_pool=None, max_len=None, live_step_len=None,
+                          **kwargs):
         input_ids = input_batch["input_ids"]
         positions = input_batch.get("positions")
         segment_ids = input_batch.get("input_segment_ids")
@@ -176,6 +177,8 @@ class Decoder(BaseLayer):
                 time_step=cached_states["time_step"], data=x, page_pool=page_pool, max_len=max_len, **tkw)
             states = {"transformer_state": states}
         else:
+            if live_step_len is not None:
+                tkw["live_step_len"] = live_step_len
             states, out = self.transformer.extend_step(
                 cached_states["transformer_state"], x, page_pool=page_pool, **tkw)
             states = {"transformer_state": states}
@@ -268,9 +271,10 @@ class Decoder(BaseLayer):
         return states, out
 
     def extend_step(self, *, cached_states: dict, input_ids: Tensor, cross_attention_data=None,
-                    cross_attention_logit_biases=None, page_pool=None):
+                    cross_attention_logit_biases=None, page_pool=None, live_step_len=None):
         """Feeds ``input_ids [B, steps]`` at positions ``time_step``..; returns
-        ``(states, {"hidden_states", "logits"})``."""
+        ``(states, {"hidden_states", "logits"})``.  ``live_step_len [B]``: valid new tokens per row
+        (stacks that support it; None: all)."""
         time_step = cached_states["time_step"]
         steps = input_ids.shape[1]
         positions = time_step[:, None] + torch.arange(steps, device=input_ids.device)[None]
@@ -278,8 +282,9 @@ class Decoder(BaseLayer):
             mode=ForwardMode.EXTEND_STEP,
             input_batch={"input_ids": input_ids, "positions": positions},
             cached_states=cached_states, cross_attention_data=cross_attention_data,
-            cross_attention_logit_biases=cross_attention_logit_biases, page_pool=page_pool)
-        states["time_step"] = time_step + steps
+            cross_attention_logit_biases=cross_attention_logit_biases, page_pool=page_pool,
+            live_step_len=live_step_len)
+        states["time_step"] = time_step + (steps if live_step_len is None else live_step_len)
         out["logits"] = self.compute_logits(out)
         return states, out
 

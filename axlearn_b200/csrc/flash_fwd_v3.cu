@@ -51,6 +51,11 @@ struct FlashFwd3Params {
   float cap_out;       // cap * log2(e); 0 = no cap    (score in log2 units = tanh(z) * cap_out)
   int causal, q_offset, window;  // window < 0: none; else keys older than row_pos - window are hidden
   int* status;
+  // Gated window attention (kGated) only: q, k, v and the gate are columns of one packed projection.
+  const void* gate;    // first gate column of row 0, or null
+  int64_t gate_ld, out_ld;
+  int vdim, every, bias;
+  float coef;          // query temperature 1 + coef * ln(floor((pos + 1) / every) + 1)
 };
 
 template <int H>
@@ -121,7 +126,10 @@ __device__ __forceinline__ void exp2_batch8(const uint32_t* s, uint64_t sc2, uin
 // kGeneral: segment ids / sliding window / logit cap are honoured (every tile takes the masking
 // path when segment ids are present).  The plain instantiation only masks diagonal and ragged
 // tiles.
-template <int H, bool kGeneral>
+// kGated (with kGeneral): scores are scaled per query row (scale * temperature), a linear distance
+// bias is taken off, and the output is multiplied by sigmoid(gate).  Head sizes up to H: the tensor
+// maps of q, k and v have the real head size as inner extent, so TMA fills the rest with zeros.
+template <int H, bool kGeneral, bool kGated = false>
 __global__ void __launch_bounds__(kF3Threads, 1)
 flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                   const __grid_constant__ CUtensorMap tmap_v, FlashFwd3Params p) {
@@ -343,6 +351,14 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       }
     }
     const uint32_t c_span = static_cast<uint32_t>(c_hi - c_lo);
+    // kGated: scores go to log2 units at once, s * row_scale + (key - query) * slope.
+    float row_scale = 1.f, slope = 0.f;
+    if (kGated) {
+      row_scale = p.sc;
+      if (p.coef != 0.f) row_scale *= 1.f + p.coef * logf(static_cast<float>((row_pos + 1) / p.every) + 1.f);
+      if (p.bias) slope = exp2f(-8.f * (head + 1) / p.N) * 1.4426950408889634f;
+    }
+    const float sc = kGated ? 1.f : p.sc;
     float m_ref = -INFINITY, l_sum = 0.f;
     bool ok = true;
     for (int it = my_lo; it < my_hi && ok; ++it) {
@@ -357,7 +373,22 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       auto mask_scores = [&](int hh, uint32_t (&r)[32]) {
         const int c0 = s0 + hh * 32;
         const uint32_t ninf = __float_as_uint(-INFINITY);
-        if (kGeneral) {
+        if (kGated) {
+          const uint64_t rs2 = f32x2(row_scale, row_scale), sl2 = f32x2(slope, slope);
+          const float d0 = static_cast<float>(c0 - row_pos);
+#pragma unroll
+          for (int j = 0; j < 32; j += 2) {
+            float x, y;
+            f32x2_split(fma2(f32x2(__uint_as_float(r[j]), __uint_as_float(r[j + 1])), rs2,
+                             fma2(add2(f32x2(d0, d0), f32x2(j, j + 1)), sl2, f32x2(0.f, 0.f))), x, y);
+            r[j] = __float_as_uint(x), r[j + 1] = __float_as_uint(y);
+          }
+          if ((c0 < c_lo) || (c0 + 31 > c_hi)) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (static_cast<uint32_t>(c0 + j - c_lo) > c_span || c_hi < c_lo) r[j] = ninf;
+          }
+        } else if (kGeneral) {
           if (p.cap_out != 0.f) {
 #pragma unroll
             for (int j = 0; j < 32; ++j)
@@ -414,7 +445,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         ok = false;
         break;
       }
-      tmax = fmaxf(tmax, other) * p.sc;  // sc > 0, so max commutes with scaling
+      tmax = fmaxf(tmax, other) * sc;  // sc > 0, so max commutes with scaling
       float alpha = 1.f;
       bool rescale = false;
       if (tmax > m_ref + 8.f) {
@@ -444,7 +475,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       // probabilities overlay the first 32 columns of its OWN 64 score columns (the chunk being
       // written was consumed just before, the other chunk lies beyond), so the two halves of a
       // row never touch each other's columns.
-      const uint64_t sc2 = f32x2(p.sc, p.sc), nm2 = f32x2(-m_use, -m_use);
+      const uint64_t sc2 = f32x2(sc, sc), nm2 = f32x2(-m_use, -m_use);
       uint64_t acc0 = f32x2(0.f, 0.f), acc1 = acc0;   // row sums, two lanes each
       auto write_probs = [&](int hh, const uint32_t (&r)[32]) {
         uint32_t q[16];
@@ -481,7 +512,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     ex_sum[(x * 2 + half) * 128 + r_in] = l_sum;
     pair_barrier(bar_id);
     l_sum += ex_sum[(x * 2 + (half ^ 1)) * 128 + r_in];
-    if (ok && row < p.T) {
+    if (!kGated && ok && row < p.T) {
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) +
                             ((static_cast<int64_t>(batch) * p.T + row) * p.N + head) * H + half * (H / 2);
       if (half == 0) {
@@ -492,7 +523,40 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         for (int c = 0; c < H / 2; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
       }
     }
-    if (ok && nt > 0) {
+    if (kGated && ok && nt > 0) {
+      const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      const int64_t tok = static_cast<int64_t>(batch) * p.T + row;
+      __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + tok * p.out_ld + head * p.vdim;
+      const __nv_bfloat16* grow = reinterpret_cast<const __nv_bfloat16*>(p.gate) + tok * p.gate_ld + head * p.vdim;
+#pragma unroll 1
+      for (int c = 0; c < H / 2; c += 16) {
+        const int col = half * (H / 2) + c;
+        uint32_t o[16];
+        tmem_ld_32x16(o_addr + c, o);
+        tmem_ld_wait();
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          if (row < p.T && col + 8 * g < p.vdim) {  // vdim is a multiple of 8
+            uint4 gate = make_uint4(0, 0, 0, 0);
+            if (p.gate != nullptr) gate = *reinterpret_cast<const uint4*>(grow + col + 8 * g);
+            const uint32_t gw[4] = {gate.x, gate.y, gate.z, gate.w};
+            uint32_t v[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+              float a = __uint_as_float(o[8 * g + 2 * u]) * inv_l, b = __uint_as_float(o[8 * g + 2 * u + 1]) * inv_l;
+              if (p.gate != nullptr) {
+                const float2 z = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162&>(gw[u]));
+                a *= 1.f / (1.f + __expf(-z.x));
+                b *= 1.f / (1.f + __expf(-z.y));
+              }
+              v[u] = pack_bf16x2(a, b);
+            }
+            *reinterpret_cast<uint4*>(orow + col + 8 * g) = make_uint4(v[0], v[1], v[2], v[3]);
+          }
+        }
+      }
+    }
+    if (!kGated && ok && nt > 0) {
       const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) +
                             ((static_cast<int64_t>(batch) * p.T + row) * p.N + head) * H + half * (H / 2);
@@ -577,13 +641,30 @@ __global__ void seg_tile_ranges_kernel(const int* __restrict__ q_seg, const int*
   }
 }
 
-template <int H, bool kGeneral>
+// Heads of `h` columns starting at column 0 of rows `ld` elements apart.
+static int make_packed_map(CUtensorMap* map, const void* base, int B, int L, int N, int h, int64_t ld) {
+  uint64_t dims[4] = {static_cast<uint64_t>(h), static_cast<uint64_t>(N), static_cast<uint64_t>(L),
+                      static_cast<uint64_t>(B)};
+  uint64_t strides[3] = {static_cast<uint64_t>(h) * 2, static_cast<uint64_t>(ld) * 2,
+                         static_cast<uint64_t>(L) * ld * 2};
+  uint32_t box[4] = {64, 1, 128, 1};
+  return make_tensor_map(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box,
+                         CU_TENSOR_MAP_SWIZZLE_128B);
+}
+
+template <int H, bool kGeneral, bool kGated = false>
 static int launch_flash_fwd3(const void* q, const void* k, const void* v, FlashFwd3Params p, cudaStream_t stream) {
   CUtensorMap tq, tk, tv;
-  if (make_bthd_map(&tq, q, p.B, p.T, p.N, H, 128)) return -2;
-  if (make_bthd_map(&tk, k, p.B, p.S, p.Nkv, H, 128)) return -2;
-  if (make_bthd_map(&tv, v, p.B, p.S, p.Nkv, H, 128)) return -2;
-  auto kernel = flash_fwd3_kernel<H, kGeneral>;
+  if (kGated) {
+    if (make_packed_map(&tq, q, p.B, p.T, p.N, p.H, p.gate_ld)) return -2;
+    if (make_packed_map(&tk, k, p.B, p.S, p.Nkv, p.H, p.gate_ld)) return -2;
+    if (make_packed_map(&tv, v, p.B, p.S, p.Nkv, p.vdim, p.gate_ld)) return -2;
+  } else {
+    if (make_bthd_map(&tq, q, p.B, p.T, p.N, H, 128)) return -2;
+    if (make_bthd_map(&tk, k, p.B, p.S, p.Nkv, H, 128)) return -2;
+    if (make_bthd_map(&tv, v, p.B, p.S, p.Nkv, H, 128)) return -2;
+  }
+  auto kernel = flash_fwd3_kernel<H, kGeneral, kGated>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, F3Smem<H>::kTotal) != cudaSuccess)
@@ -641,9 +722,36 @@ extern "C" int axb_flash_fwd_v3(const void* q, const void* k, const void* v, voi
   p.q_offset = S - T;
   p.window = window;
   p.status = status;
+  p.gate = nullptr, p.gate_ld = 0, p.out_ld = 0, p.vdim = H, p.every = 1, p.bias = 0, p.coef = 0.f;
   const bool general = q_seg != nullptr || window >= 0 || logit_cap > 0.f;
   if (H == 128) {
     return general ? launch_flash_fwd3<128, true>(q, k, v, p, stream) : launch_flash_fwd3<128, false>(q, k, v, p, stream);
   }
   return general ? launch_flash_fwd3<64, true>(q, k, v, p, stream) : launch_flash_fwd3<64, false>(q, k, v, p, stream);
+}
+
+// Gated sliding-window attention of whole prompts (positions from 0), see window_attn.cu for the formula.
+// q / k / v / gate point at their first column in a packed projection [B, T, ld] (bf16); out [B, T, out_ld],
+// head h at column h * vdim.  Head sizes are multiples of 8 up to 128, as are ld, out_ld and the column
+// offsets (16-byte alignment).  gate may be null, coef 0 (no temperature), bias 0 (no distance bias).
+extern "C" int axb_flash_fwd_gated(const void* q, const void* k, const void* v, const void* gate, void* out, int B,
+                                   int T, int N, int Nkv, int dim, int vdim, int64_t ld, int64_t out_ld, float scale,
+                                   int window, float coef, int every, int bias, int* status, cudaStream_t stream) {
+  using namespace axb;
+  if (N % Nkv != 0 || dim > 128 || vdim > 128 || (dim % 8) || (vdim % 8) || (ld % 8) || (out_ld % 8) || window < 1 ||
+      every < 1 || out_ld < static_cast<int64_t>(N) * vdim)
+    return -10;
+  const uintptr_t align = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) |
+                          reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(gate) |
+                          reinterpret_cast<uintptr_t>(out);
+  if (align & 15) return -10;
+  FlashFwd3Params p;
+  p.out = out, p.lse = nullptr;
+  p.q_seg = nullptr, p.k_seg = nullptr, p.ranges = nullptr;
+  p.B = B, p.T = T, p.S = T, p.N = N, p.Nkv = Nkv, p.H = dim;
+  p.sc = scale * 1.4426950408889634f, p.cap_in = 0.f, p.cap_out = 0.f;
+  p.causal = 1, p.q_offset = 0, p.window = window - 1, p.status = status;
+  p.gate = gate, p.gate_ld = ld, p.out_ld = out_ld, p.vdim = vdim, p.every = every, p.bias = bias, p.coef = coef;
+  if (dim <= 64 && vdim <= 64) return launch_flash_fwd3<64, true, true>(q, k, v, p, stream);
+  return launch_flash_fwd3<128, true, true>(q, k, v, p, stream);
 }

@@ -1,4 +1,5 @@
-"""Decode engine for Fuji-style decoders: paged KV cache, tensor parallelism, CUDA-graph steps.
+"""Decode engines: Fuji-style decoders (paged KV cache, tensor parallelism) and any decoder whose
+layers keep their states in place, both as CUDA-graph steps on persistent buffers.
 
 What the reference does for generation is a jitted ``while_loop`` over ``Decoder.extend_step``
 (axlearn/common/decoder.py:286-448, axlearn/common/decoding.py:978-1150) with a functional KV
@@ -34,6 +35,7 @@ from typing import Any, Optional
 
 import torch
 
+from axlearn_b200.common.utils import flatten_items
 from axlearn_b200.ops import attention_ops, cuda_ops, decode_ops
 
 Tensor = torch.Tensor
@@ -113,15 +115,100 @@ def weights_from_fuji_state(model_state: dict, dims: FujiDims, *, rank: int = 0,
     return {"layers": layers, "emb": emb, "head": head, "final_norm": put(_get(dec, "output_norm/scale"))}
 
 
-class DecodeEngine:
+class BaseDecodeEngine:
+    """Batch decoding on persistent buffers: subclasses provide ``prefill`` and ``_step``; this class owns
+    the token / length / logits buffers, the captured step and the loops over it.
+
+    ``_step`` consumes ``self.tokens`` (the latest token of every sequence), leaves fp32 logits in
+    ``self.logits`` and the greedy pick in ``self.tokens``, and touches nothing but persistent buffers."""
+
+    def __init__(self, *, batch: int, vocab_size: int, device, use_graph: bool):
+        self.batch, self.device = batch, torch.device(device)
+        self.lengths = torch.zeros(batch, dtype=torch.int32, device=self.device)
+        self.tokens = torch.zeros(batch, dtype=torch.int64, device=self.device)
+        # Logits of the latest position (a fixed buffer: the captured step writes into it, and a
+        # sampler outside the graph reads it).
+        self.logits = torch.zeros(batch, vocab_size, dtype=torch.float32, device=self.device)
+        self._use_graph = use_graph and self.device.type == "cuda"
+        self._graph: Optional[torch.cuda.CUDAGraph] = None
+        self.launches_per_step = 0
+
+    def prefill(self, prompt_ids: Tensor, lengths: Optional[Tensor] = None) -> Tensor:
+        raise NotImplementedError(type(self))
+
+    def _step(self) -> None:
+        raise NotImplementedError(type(self))
+
+    def _mutable_buffers(self) -> list:
+        """Buffers a step changes and that a warm-up step must leave as they were."""
+        return [self.lengths, self.tokens]
+
+    def _check_status(self) -> None:
+        if self.device.type == "cuda":
+            cuda_ops.check_status(self.device)
+
+    @torch.no_grad()
+    def decode(self, steps: int) -> Tensor:
+        """Generates ``steps`` further tokens per sequence (after ``prefill``); returns them
+        ``[batch, steps]``.  The first call captures the step in a CUDA graph."""
+        out = torch.empty((self.batch, steps), dtype=torch.int64, device=self.device)
+        self._ensure_graph()
+        for i in range(steps):
+            if self._graph is not None:
+                self._graph.replay()
+            else:
+                self._step()
+            out[:, i] = self.tokens
+        self._check_status()
+        return out
+
+    def _ensure_graph(self) -> None:
+        if self._use_graph and self._graph is None:
+            # Warm up on a side stream (lazy module loading, tensor-map encoding), restoring
+            # the state the warm-up step consumed, then capture (capturing executes nothing).  The
+            # epoch of a tensor-parallel all-reduce keeps counting: peers warm up the same number of steps.
+            buffers = self._mutable_buffers()
+            saved = [t.clone() for t in buffers]
+            s = torch.cuda.Stream(device=self.device)
+            s.wait_stream(torch.cuda.current_stream(self.device))
+            with torch.cuda.stream(s):
+                self._step()
+            torch.cuda.current_stream(self.device).wait_stream(s)
+            for t, old in zip(buffers, saved):
+                t.copy_(old)
+            self._graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(self._graph):
+                self._step()
+
+    @torch.no_grad()
+    def step_logits(self, tokens: Tensor) -> Tensor:
+        """Feeds one token per sequence (``[batch]``: the token at each sequence's current end),
+        appends its K/V and returns the fp32 logits of the next position ``[batch, vocab]`` -- the
+        engine as a ``tokens -> scores`` function for samplers and searches that live outside."""
+        self._ensure_graph()
+        self.tokens.copy_(tokens.reshape(-1))
+        if self._graph is not None:
+            self._graph.replay()
+        else:
+            self._step()
+        return self.logits
+
+    @torch.no_grad()
+    def generate(self, prompt_ids: Tensor, max_new_tokens: int) -> Tensor:
+        first = self.prefill(prompt_ids)
+        rest = self.decode(max_new_tokens - 1) if max_new_tokens > 1 else first[:, :0]
+        return torch.cat([first[:, None], rest], dim=1)
+
+
+class DecodeEngine(BaseDecodeEngine):
     """Greedy generation for ``batch`` sequences of up to ``max_len`` tokens on one GPU of a
     tensor-parallel group (``group=None``: single GPU)."""
 
     def __init__(self, weights: dict, dims: FujiDims, *, batch: int, max_len: int, page_size: int = 16,
                  group=None, device=None, use_graph: bool = True, prefill_chunk_tokens: int = 16384):
-        self.w, self.dims = weights, dims
-        self.batch, self.page_size = batch, page_size
-        self.device = device if device is not None else weights["emb"].device
+        super().__init__(batch=batch, vocab_size=dims.vocab_size, use_graph=use_graph,
+                         device=device if device is not None else weights["emb"].device)
+        self.w, self.dims, self.page_size = weights, dims, page_size
         self.group = group
         if group is not None:
             import torch.distributed as dist
@@ -139,11 +226,6 @@ class DecodeEngine:
         self.v_pools = [torch.zeros(pool, dtype=torch.bfloat16, device=self.device) for _ in range(d.num_layers)]
         self.page_table = torch.arange(batch * self.max_pages, dtype=torch.int32, device=self.device).reshape(
             batch, self.max_pages)
-        self.lengths = torch.zeros(batch, dtype=torch.int32, device=self.device)
-        self.tokens = torch.zeros(batch, dtype=torch.int64, device=self.device)
-        # Logits of the latest position (a fixed buffer: the captured step writes into it, and a
-        # sampler outside the graph reads it).
-        self.logits = torch.zeros(batch, dims.vocab_size, dtype=torch.float32, device=self.device)
         self.splits = decode_ops.default_splits(batch, self.nkv_l, self.nq_l // self.nkv_l, self.max_len, page_size)
         self._scratch = torch.empty(
             max(1, decode_ops._lib().axb_decode_attn_scratch_floats(batch, self.nq_l, self.splits)),  # pylint: disable=protected-access
@@ -153,10 +235,7 @@ class DecodeEngine:
         if self.world > 1:
             self._allreduce = decode_ops.OneShotAllReduce(
                 batch * d.hidden_dim, 2 * d.num_layers, group=group, device=self.device)
-        self._use_graph = use_graph
-        self._graph: Optional[torch.cuda.CUDAGraph] = None
         self._prefill_chunk_tokens = prefill_chunk_tokens
-        self.launches_per_step = 0
 
     # ------------------------------------------------------------------ shared pieces
     def _gemm_reduce(self, a: Tensor, w: Tensor, residual: Tensor, site: int) -> Tensor:
@@ -228,8 +307,7 @@ class DecodeEngine:
             self.lengths.copy_(lengths.to(self.lengths.dtype))
         self.logits.copy_(self._logits(last_hidden))
         self.tokens.copy_(self.logits.argmax(dim=-1))
-        if self.device.type == "cuda":
-            cuda_ops.check_status(self.device)
+        self._check_status()
         return self.tokens.clone()
 
     def _logits(self, hidden: Tensor) -> Tensor:
@@ -270,59 +348,109 @@ class DecodeEngine:
         self.tokens.copy_(self.logits.argmax(dim=-1))
         self.launches_per_step = cuda_ops.launch_count - before
 
+
+class ModuleDecodeEngine(BaseDecodeEngine):
+    """The engine over any ``Decoder`` whose stack keeps its states in place (``GRAPH_DECODE``): prompts go
+    through ``Decoder.prefill_states``, the decoding step is ``Decoder.extend_step`` captured in a CUDA
+    graph -- the layers themselves are the implementation, there is no second one here.
+
+    ``params`` is the decoder's parameter tree.  Rows can be taken out of a step (``set_active``): their
+    states and lengths stay as they are."""
+
+    def __init__(self, decoder, params: dict, *, batch: int, max_len: int, dtype: torch.dtype = torch.bfloat16,
+                 device=None, use_graph: bool = True, prefill_chunk_tokens: int = 65536):
+        cfg = decoder.config
+        super().__init__(batch=batch, vocab_size=cfg.vocab_size, use_graph=use_graph, device=device)
+        self.decoder, self.params, self.max_len = decoder, params, max_len
+        self.active = torch.ones(batch, dtype=torch.int32, device=self.device)
+        self._dtype, self._prefill_chunk_tokens = dtype, prefill_chunk_tokens
+        self.states = self._call("init_states", batch_size=batch, max_sequence_length=max_len, dtype=dtype,
+                                 device=self.device)
+
+    def _call(self, method: str, **inputs):
+        from axlearn_b200.common.module import functional
+
+        return functional(self.decoder, None, self.params, inputs, method=method, is_training=False)[0]
+
+    def _mutable_buffers(self) -> list:
+        return super()._mutable_buffers() + [t for _, t in flatten_items(self.states)]
+
+    def set_active(self, rows: Tensor) -> None:
+        """``rows [batch]``: nonzero = takes part in the following steps."""
+        self.active.copy_(rows)
+
     @torch.no_grad()
-    def decode(self, steps: int) -> Tensor:
-        """Generates ``steps`` further tokens per sequence (after ``prefill``); returns them
-        ``[batch, steps]``.  The first call captures the step in a CUDA graph."""
-        out = torch.empty((self.batch, steps), dtype=torch.int64, device=self.device)
-        self._ensure_graph()
-        for i in range(steps):
-            if self._graph is not None:
-                self._graph.replay()
-            else:
-                self._step()
-            out[:, i] = self.tokens
-        cuda_ops.check_status(self.device)
+    def prefill(self, prompt_ids: Tensor, lengths: Optional[Tensor] = None,
+                logits_at: Optional[tuple] = None) -> Tensor:
+        """Runs right-padded prompts ``[batch, T]`` from empty states and returns the greedy first token of
+        every sequence (logits of the last position in ``self.logits``).  ``logits_at = (rows, positions)``
+        returns the fp32 logits ``[n, vocab]`` of those places instead."""
+        b, t = prompt_ids.shape
+        assert b == self.batch and t <= self.max_len, (prompt_ids.shape, self.batch, self.max_len)
+        if lengths is None:
+            lengths = torch.full((b,), t, dtype=torch.int32)
+        lengths = lengths.to(device=self.device, dtype=torch.int32)
+        prompt_ids = prompt_ids.to(self.device)
+        per_chunk = max(1, self._prefill_chunk_tokens // t)
+        last, picked = [], []
+        for b0 in range(0, b, per_chunk):
+            b1 = min(b, b0 + per_chunk)
+            states, out = self._call("prefill_states", time_step=lengths[b0:b1],
+                                     input_batch={"input_ids": prompt_ids[b0:b1]}, max_sequence_length=self.max_len)
+            hidden = out["hidden_states"]
+            for (_, mine), (_, new) in zip(flatten_items(self.states), flatten_items(states)):
+                mine[b0:b1].copy_(new)
+            rows = torch.arange(b1 - b0, device=self.device)
+            last.append(hidden[rows, (lengths[b0:b1].long() - 1).clamp(min=0)])
+            if logits_at is not None:
+                at_rows, at_pos = (x.to(self.device).long() for x in logits_at)
+                inside = torch.nonzero((at_rows >= b0) & (at_rows < b1))[:, 0]
+                picked.append((inside, hidden[at_rows[inside] - b0, at_pos[inside]]))
+        self.lengths.copy_(lengths)
+        self.logits.copy_(self._logits(torch.cat(last)))
+        self.tokens.copy_(self.logits.argmax(dim=-1))
+        if logits_at is None:
+            self._check_status()
+            return self.tokens.clone()
+        order = torch.cat([i for i, _ in picked])
+        rows = torch.cat([h for _, h in picked])[torch.argsort(order)]
+        out = self._logits(rows) if len(rows) else rows.new_zeros((0, self.logits.shape[1]), dtype=torch.float32)
+        self._check_status()
         return out
 
-    def _ensure_graph(self) -> None:
-        if self._use_graph and self._graph is None:
-            # Warm up on a side stream (lazy module loading, tensor-map encoding), restoring
-            # the state the warm-up steps consumed, then capture.
-            saved = (self.lengths.clone(), self.tokens.clone())
-            epoch = None if self._allreduce is None else self._allreduce.epoch.clone()
-            s = torch.cuda.Stream(device=self.device)
-            s.wait_stream(torch.cuda.current_stream(self.device))
-            with torch.cuda.stream(s):
-                self._step()
-            torch.cuda.current_stream(self.device).wait_stream(s)
-            self.lengths.copy_(saved[0])
-            self.tokens.copy_(saved[1])
-            del epoch  # The epoch keeps counting: peers warmed up the same number of steps.
-            self._graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(self._graph):
-                self._step()
-            self.lengths.copy_(saved[0])
-            self.tokens.copy_(saved[1])
+    def _logits(self, hidden: Tensor) -> Tensor:
+        return self._call("compute_logits", forward_outputs={"hidden_states": hidden}).float()
 
     @torch.no_grad()
-    def step_logits(self, tokens: Tensor) -> Tensor:
-        """Feeds one token per sequence (``[batch]``: the token at each sequence's current end),
-        appends its K/V and returns the fp32 logits of the next position ``[batch, vocab]`` -- the
-        engine as a ``tokens -> scores`` function for samplers and searches that live outside."""
-        self._ensure_graph()
-        self.tokens.copy_(tokens.reshape(-1))
-        if self._graph is not None:
-            self._graph.replay()
-        else:
-            self._step()
-        return self.logits
+    def extend(self, token_ids: Tensor, live: Optional[Tensor] = None) -> Tensor:
+        """Feeds ``[batch, steps]`` further tokens (``live [batch]`` valid ones per row) after what every
+        sequence has seen; returns the fp32 logits ``[batch, steps, vocab]``."""
+        b, steps = token_ids.shape
+        live = torch.full((b,), steps, dtype=torch.int32) if live is None else live
+        live = live.to(device=self.device, dtype=torch.int32)
+        states, out = self._call("extend_step", cached_states=self.states, input_ids=token_ids.to(self.device),
+                                 live_step_len=live)
+        self._keep(states)
+        self.lengths.add_(live)
+        logits = out["logits"].float()
+        self.logits.copy_(logits[torch.arange(b, device=self.device), (live.long() - 1).clamp(min=0)])
+        self._check_status()
+        return logits
 
-    @torch.no_grad()
-    def generate(self, prompt_ids: Tensor, max_new_tokens: int) -> Tensor:
-        first = self.prefill(prompt_ids)
-        rest = self.decode(max_new_tokens - 1) if max_new_tokens > 1 else first[:, :0]
-        return torch.cat([first[:, None], rest], dim=1)
+    def _keep(self, states: dict) -> None:
+        for (_, mine), (_, new) in zip(flatten_items(self.states), flatten_items(states)):
+            if mine.data_ptr() != new.data_ptr():
+                mine.copy_(new)
+
+    def _step(self) -> None:
+        before = cuda_ops.launch_count
+        states, out = self._call("extend_step", cached_states=self.states, input_ids=self.tokens[:, None],
+                                 live_step_len=self.active)
+        self._keep(states)
+        self.lengths.add_(self.active)
+        self.logits.copy_(out["logits"][:, -1])
+        self.tokens.copy_(self.logits.argmax(dim=-1))
+        self.launches_per_step = cuda_ops.launch_count - before
 
 
 # ------------------------------------------------------------------------------------------
@@ -362,7 +490,7 @@ def dims_from_decoder(decoder) -> Optional[FujiDims]:
         return None
 
 
-def engine_for_decoder(decoder, *, batch: int, max_len: int) -> Optional["DecodeEngine"]:
+def engine_for_decoder(decoder, *, batch: int, max_len: int) -> Optional[BaseDecodeEngine]:
     """A (cached) engine over the decoder's current parameters, or None when the decoder, its
     placement or its shapes are outside what the engine implements."""
     from axlearn_b200.parallel.mesh import current_mesh
@@ -372,10 +500,20 @@ def engine_for_decoder(decoder, *, batch: int, max_len: int) -> Optional["Decode
     mesh = current_mesh()
     if mesh is not None and mesh.size > 1:
         return None
+    state = decoder.parameter_tree()
+    if getattr(decoder.config.transformer.klass, "GRAPH_DECODE", False):
+        emb = _get(state, "emb/token_emb/weight")
+        if not emb.is_cuda or emb.dtype not in (torch.bfloat16, torch.float32):
+            return None
+        key = (id(decoder), batch, max_len, emb.data_ptr())
+        if key not in _ENGINES:
+            _ENGINES.clear()
+            _ENGINES[key] = ModuleDecodeEngine(decoder, state, batch=batch, max_len=max_len, dtype=emb.dtype,
+                                               device=emb.device)
+        return _ENGINES[key]
     dims = dims_from_decoder(decoder)
     if dims is None or dims.head_dim != 128:
         return None
-    state = decoder.parameter_tree()
     emb = _get(state, "emb/token_emb/weight")
     if not emb.is_cuda or emb.dtype != torch.bfloat16:
         return None

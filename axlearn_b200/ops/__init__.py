@@ -11,6 +11,7 @@ from axlearn_b200.ops.dispatch import (  # noqa: F401
     attention,
     cross_entropy,
     linear,
+    linear_f32,
     lm_head_cross_entropy,
     add_rms_norm,
     rms_norm,

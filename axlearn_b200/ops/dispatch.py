@@ -138,6 +138,15 @@ def linear(x, w):
     return _LinearKept.apply(x, w, y)
 
 
+def linear_f32(x, w):
+    """``x[..., K] @ w[K, N]`` with an fp32 result (the accumulators as they are): output heads."""
+    if _cuda(x, w) and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and not (
+            torch.is_grad_enabled() and (x.requires_grad or w.requires_grad)):
+        y = _ops().gemm(x.reshape(-1, x.shape[-1]), w, out_dtype=torch.float32)
+        return y.reshape(x.shape[:-1] + (w.shape[1],))
+    return linear(x, w).float()
+
+
 def attention(
     q,
     k,
