@@ -58,6 +58,10 @@ def _args():
                     "(the product of the sizes must be --gpus; the batch is per data-parallel rank)")
     ap.add_argument("--kernel_table", default=None, help="after the timed regions, profile two more steps with the "
                     "torch profiler and write per-kernel device-time shares to this file (rank 0)")
+    ap.add_argument("--serving", action="store_true", help="non-headline: prefill and decode throughput of the Sagisun "
+                    "design beside the Fuji decoder of equal widths, one JSON line per (size, model, batch)")
+    ap.add_argument("--serving_sizes", default=None, help="--serving: comma-separated subset of the sizes")
+    ap.add_argument("--serving_table", default=None, help="--serving: write per-kernel device times to this file")
     ap.add_argument("--skip_parity", action="store_true", help="N>1: skip the one-step fused-vs-library parity record")
     return ap.parse_args()
 
@@ -128,6 +132,16 @@ def main():
             "unavailable": "apple/axlearn needs jax/jaxlib(cuda12)/tensorstore/optax wheels and the hatchling "
                            "build backend; none are in the offline wheelhouse, so it cannot be installed",
         }))
+        return
+    if args.serving:
+        from axlearn_b200.inference import bench_serving
+
+        sampler = ClockSampler(0)
+        sampler.start()
+        bench_serving.run(steps=args.steps, warmup=args.warmup, table=args.serving_table,
+                          sizes=args.serving_sizes.split(",") if args.serving_sizes else None,
+                          emit=lambda line: print(line, flush=True))
+        print(json.dumps({"clocks": sampler.stop()}))
         return
 
     import torch
