@@ -55,6 +55,16 @@ class PaddedLinear(BaseLayer):
         return ops.linear(x, self.parameters["weight"].to(x.dtype).t())
 
 
+_side_streams: dict = {}
+
+
+def _side_stream(device: torch.device) -> "torch.cuda.Stream":
+    index = device.index if device.index is not None else torch.cuda.current_device()
+    if index not in _side_streams:
+        _side_streams[index] = torch.cuda.Stream(device=index)
+    return _side_streams[index]
+
+
 class BaseSequenceMixer(BaseLayer):
     @config_class
     class Config(BaseLayer.Config):
@@ -232,10 +242,23 @@ class ParallelMixer(BaseLayer):
     def forward(self, x: Tensor, *, start=None, live=None, state=None):
         proj = self.i_proj(x)
         outs, states = {}, {}
-        for side in ("left", "right"):
-            mixer = getattr(self, side)
-            outs[side], states[side] = mixer.mix(proj, self._columns[side], start=start, live=live,
-                                                 state=None if state is None else state[side])
+
+        def mix(side):
+            outs[side], states[side] = getattr(self, side).mix(
+                proj, self._columns[side], start=start, live=live, state=None if state is None else state[side])
+
+        if x.is_cuda and x.shape[1] == 1 and not torch.is_grad_enabled():
+            # A decoding step's kernels are small: the two mixers run next to each other.  (The side stream's
+            # tensors are read before the next fork, which orders their reuse.)
+            main, side_stream = torch.cuda.current_stream(x.device), _side_stream(x.device)
+            side_stream.wait_stream(main)
+            with torch.cuda.stream(side_stream):
+                mix("right")
+            mix("left")
+            main.wait_stream(side_stream)
+        else:
+            mix("left")
+            mix("right")
         p = self.parameters
         pair = hyper_ops.NormedPair(outs["left"], outs["right"], p["left_norm_scale"], p["right_norm_scale"],
                                     self._config.norm_eps)

@@ -374,14 +374,16 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const int c0 = s0 + hh * 32;
         const uint32_t ninf = __float_as_uint(-INFINITY);
         if (kGated) {
-          const uint64_t rs2 = f32x2(row_scale, row_scale), sl2 = f32x2(slope, slope);
-          const float d0 = static_cast<float>(c0 - row_pos);
+          // The distance term of a pair of keys advances by addition (two-wide, like the scaling).
+          const uint64_t rs2 = f32x2(row_scale, row_scale), step2 = f32x2(2.f * slope, 2.f * slope);
+          const float d0 = static_cast<float>(c0 - row_pos) * slope;
+          uint64_t bias2 = f32x2(d0, d0 + slope);
 #pragma unroll
           for (int j = 0; j < 32; j += 2) {
             float x, y;
-            f32x2_split(fma2(f32x2(__uint_as_float(r[j]), __uint_as_float(r[j + 1])), rs2,
-                             fma2(add2(f32x2(d0, d0), f32x2(j, j + 1)), sl2, f32x2(0.f, 0.f))), x, y);
+            f32x2_split(fma2(f32x2(__uint_as_float(r[j]), __uint_as_float(r[j + 1])), rs2, bias2), x, y);
             r[j] = __float_as_uint(x), r[j + 1] = __float_as_uint(y);
+            bias2 = add2(bias2, step2);
           }
           if ((c0 < c_lo) || (c0 + 31 > c_hi)) {
 #pragma unroll

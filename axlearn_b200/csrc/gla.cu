@@ -32,7 +32,7 @@ struct GlaArgs {
   void* out;             // [B, T, out_ld]
   float* o_raw;          // [B, T, heads, vdim] un-normalised outputs (multi-slice, scan)
   float* seg_state;      // [B, heads, segments, dim, vdim] (segmented runs)
-  float* seg_decay;      // [B, heads, segments, dim]
+  float* seg_decay;      // [B, heads, segments, dim], log2
   const int* start;
   const int* live;
   int64_t ld, out_ld;
@@ -251,8 +251,9 @@ __global__ void gla_norm_gate_kernel(GlaArgs a) {
 //   q^_i = q_i exp(G_i)      k~_j = k_j exp(-G_j)
 //   o_i  = S_in^T q^_i + sum_{j <= i} (q^_i . k~_j) v_j
 //   S_out = diag(exp(G_64)) (S_in + sum_j k~_j v_j^T)
+// (the code keeps G in base 2).
 // The factored form is exact as long as exp(-G_64) stays finite: a chunk with a channel whose total
-// decay exceeds e^-60 is run token by token on the same register state instead (a uniform branch).
+// decay exceeds 2^-86 is run token by token on the same register state instead (a uniform branch).
 //
 // What enters the recurrence is kept to fp32 accuracy: k~, the scores and the state as matrix operands
 // are split into two bf16 terms (hi + lo); q^ is one bf16, like the projection q itself.
@@ -298,32 +299,57 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 __device__ __forceinline__ void cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sptr(dst)), "l"(src) : "memory");
 }
+__device__ __forceinline__ void prefetch_row(const __nv_bfloat16* p, int n) {
+  for (int c = 0; c < n; c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + c));
+}
 __device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// 64 rows of `n` elements (source pitch ld) into a tile of W columns, zero beyond n and beyond `rows`.
+// 64 rows of `n` elements (source pitch ld) into a tile of W columns, zero beyond n and beyond `rows`.  A
+// thread keeps its column and walks the rows.
 template <int W>
 __device__ __forceinline__ void load_tile(__nv_bfloat16* tile, int pitch, const __nv_bfloat16* src, int64_t ld, int n,
                                           int rows, bool vec) {
-  for (int i = threadIdx.x; i < kGcTok * (W / 8); i += kGcThreads) {
-    const int r = i / (W / 8), c = (i % (W / 8)) * 8;
-    __nv_bfloat16* dst = tile + r * pitch + c;
-    if (vec && r < rows && c + 8 <= n) {
-      cp16(dst, src + r * ld + c);
-    } else {
+  constexpr int kPer = W / 8, kStep = kGcThreads / kPer;
+  const int c = (threadIdx.x % kPer) * 8, r0 = threadIdx.x / kPer;
+  __nv_bfloat16* dst = tile + r0 * pitch + c;
+  const __nv_bfloat16* p = src + r0 * ld + c;
+  const bool whole = vec && c + 8 <= n;
 #pragma unroll
-      for (int e = 0; e < 8; ++e)
-        dst[e] = r < rows && c + e < n ? src[r * ld + c + e] : __float2bfloat16(0.f);
+  for (int r = r0; r < kGcTok; r += kStep) {
+    if (whole && r < rows) {
+      cp16(dst, p);
+    } else if (vec || c >= n || r >= rows) {
+      *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    } else {
+#pragma unroll 1
+      for (int e = 0; e < 8; ++e) dst[e] = c + e < n ? p[e] : __float2bfloat16(0.f);
     }
+    dst += kStep * pitch;
+    p += kStep * ld;
   }
 }
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float kLog2e = 1.4426950408889634f;
+// x * sigmoid(x)
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + ex2(-x * kLog2e)); }
 
 }  // namespace
 
 template <int DP, int VS>
 struct GcSmem {
   static constexpr int kQP = DP + 8, kVP = VS + 8, kAP = kGcTok + 8;
-  static constexpr int kQ = 0;                               // bf16 [64][kQP]  q, then q^
-  static constexpr int kK = kQ + kGcTok * kQP * 2;           // bf16            k, then k~ hi
+  static constexpr int kQ = 0;                               // bf16 [64][kQP]  q, then q^; [64][kVP] gate, then out
+  static constexpr int kK = kQ + kGcTok * (kQP > kVP ? kQP : kVP) * 2;  // bf16 k, then k~ hi
   static constexpr int kV = kK + kGcTok * kQP * 2;           // bf16 [64][kVP]
   static constexpr int kKlo = kV + kGcTok * kVP * 2;         // bf16 [64][kQP]  k~ lo   } token-by-token path:
   static constexpr int kA = kKlo + kGcTok * kQP * 2;         // bf16 2 x [64][kAP]      } fp32 decay [64][DP]
@@ -369,9 +395,19 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
   const int t_lo = seg * a.seg_tokens, t_hi = a.segments > 1 ? min(a.T, t_lo + a.seg_tokens) : a.T;
   const int vcols = min(VS, a.vdim - d0);
   const bf16* base = static_cast<const bf16*>(a.proj) + static_cast<int64_t>(b) * a.T * a.ld;
-  const bool vec = !((a.ld | a.q_off | a.k_off | a.v_off | a.dim | a.vdim) & 7);
+  const bool vec = !((a.ld | a.q_off | a.k_off | a.v_off | a.g_off | a.dim | a.vdim) & 7);
+  const bool vec_a1 = vec && !((a.a1_off | a.rank) & 7);
   const bool owner = warp < kWarpsV;
   const int v0 = warp * 16 * MV;  // first value column of this warp in the slice
+  const float inv_vdim = 1.f / a.vdim;
+  float nw[MV * 2][2];
+#pragma unroll
+  for (int n = 0; n < MV * 2; ++n)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int v = v0 + n * 8 + lc + e;
+      nw[n][e] = !kStateOnly && slices == 1 && owner && v < vcols ? a.norm_w[v] : 0.f;
+    }
 
   for (int i = tid; i < DP * rp; i += kGcThreads) {
     const int c = i / rp, r = i % rp;
@@ -380,7 +416,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
                            : __float2bfloat16(0.f);
   }
   for (int c = tid; c < DP; c += kGcThreads) {
-    sBias[c] = c < a.dim ? a.a2_bias[h * a.dim + c] : 0.f;
+    sBias[c] = c < a.dim ? a.a2_bias[h * a.dim + c] * kLog2e : 0.f;
     sSum[c] = 0.f;
   }
 
@@ -421,12 +457,35 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
     if (!kStateOnly) load_tile<DP>(sQ, L::kQP, src + a.q_off + h * a.dim, a.ld, a.dim, rows, vec);
     load_tile<DP>(sK, L::kQP, src + a.k_off + h * a.dim, a.ld, a.dim, rows, vec);
     load_tile<VS>(sV, L::kVP, src + a.v_off + h * a.vdim + d0, a.ld, vcols, rows, vec);
-    for (int i = tid; i < kGcTok * rp; i += kGcThreads) {
-      const int r = i / rp, c = i % rp;
-      sA1[r * rpp + c] = r < rows && c < a.rank ? src[r * a.ld + a.a1_off + c] : __float2bfloat16(0.f);
+    if (vec_a1) {
+      for (int i = tid; i < kGcTok * (rp / 8); i += kGcThreads) {
+        const int r = i / (rp / 8), c = (i % (rp / 8)) * 8;
+        if (r < rows && c < a.rank)
+          cp16(sA1 + r * rpp + c, src + r * a.ld + a.a1_off + c);
+        else
+          *reinterpret_cast<uint4*>(sA1 + r * rpp + c) = make_uint4(0, 0, 0, 0);
+      }
+    } else {
+      for (int i = tid; i < kGcTok * rp; i += kGcThreads) {
+        const int r = i / rp, c = i % rp;
+        sA1[r * rpp + c] = r < rows && c < a.rank ? src[r * a.ld + a.a1_off + c] : __float2bfloat16(0.f);
+      }
+    }
+    // The next chunk's rows start their way from DRAM to L2 while this one is computed.
+    if (t0 + kGcTok + (tid >> 2) < min(live, t_hi)) {
+      const bf16* next = src + (kGcTok + (tid >> 2)) * a.ld;
+      switch (tid & 3) {
+        case 0: prefetch_row(next + a.q_off + h * a.dim, kStateOnly ? 0 : a.dim); break;
+        case 1: prefetch_row(next + a.k_off + h * a.dim, a.dim); break;
+        case 2: prefetch_row(next + a.v_off + h * a.vdim + d0, vcols); break;
+        default: prefetch_row(next + a.g_off + h * a.vdim + d0, kStateOnly ? 0 : vcols); break;
+      }
     }
     cp_wait_all();
     __syncthreads();
+    auto load_gate = [&]() {  // over q^, once nobody reads it any more
+      if (!kStateOnly && slices == 1) load_tile<VS>(sQ, L::kVP, src + a.g_off + h * a.vdim, a.ld, vcols, rows, vec);
+    };
 
     // Log decays of this warp's channels [warp * DP / 8, + DP / 8): rows = tokens.
     float g[4][ZT][4];
@@ -455,16 +514,24 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
       }
 #pragma unroll
       for (int n = 0; n < ZT; ++n) {
+        // In base 2: log2 sigmoid(z) = min(z', 0) - log2(1 + 2^-|z'|), z' = z log2(e).
         const int c = warp * (DP / 8) + n * 8 + lc;
+        const float2 bias = *reinterpret_cast<const float2*>(sBias + c);
+        const float t0 = c < a.dim ? a.inv_tau : 0.f, t1 = c + 1 < a.dim ? a.inv_tau : 0.f;
 #pragma unroll
         for (int m = 0; m < 4; ++m)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const int r = m * 16 + lr + (e >> 1) * 8;
-            const float z = g[m][n][e] + sBias[c + (e & 1)];
-            const float x = fminf(z, 0.f) - __logf(1.f + __expf(-fabsf(z)));
-            g[m][n][e] = r < rows && c + (e & 1) < a.dim ? x * a.inv_tau : 0.f;
+            const float z = fmaf(g[m][n][e], kLog2e, e & 1 ? bias.y : bias.x);
+            g[m][n][e] = (fminf(z, 0.f) - lg2(1.f + ex2(-fabsf(z)))) * (e & 1 ? t1 : t0);
           }
+        if (rows < kGcTok) {
+#pragma unroll
+          for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              if (m * 16 + lr + (e >> 1) * 8 >= rows) g[m][n][e] = 0.f;
+        }
       }
     };
     log_decays();
@@ -491,14 +558,14 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
         g_end[n][e] = carry;
         worst = fminf(worst, carry);
       }
-    const bool sequential = __syncthreads_or(worst < -60.f);
+    const bool sequential = __syncthreads_or(worst < -86.f);
     if (lr == 0) {
 #pragma unroll
       for (int n = 0; n < ZT; ++n)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int c = warp * (DP / 8) + n * 8 + lc + e;
-          sEnd[c] = __expf(g_end[n][e]);
+          sEnd[c] = ex2(g_end[n][e]);
           if (kStateOnly) sSum[c] += g_end[n][e];
         }
     }
@@ -524,12 +591,12 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
             if (!kStateOnly) {
               uint32_t* pq = reinterpret_cast<uint32_t*>(sQ + r * L::kQP + c);
               const float2 q = unpack2(*pq);
-              *pq = pack2(q.x * a.q_scale * __expf(g0), q.y * a.q_scale * __expf(g1));
+              *pq = pack2(q.x * a.q_scale * ex2(g0), q.y * a.q_scale * ex2(g1));
             }
             uint32_t* pk = reinterpret_cast<uint32_t*>(sK + r * L::kQP + c);
             const float2 k = unpack2(*pk);
             uint32_t hi, lo;
-            split2(k.x * __expf(-g0), k.y * __expf(-g1), hi, lo);
+            split2(k.x * ex2(-g0), k.y * ex2(-g1), hi, lo);
             *pk = hi;
             *reinterpret_cast<uint32_t*>(sKlo + r * L::kQP + c) = lo;
           }
@@ -598,6 +665,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
           }
         }
         __syncthreads();
+        load_gate();
         if (owner) {
           // O += A V.
 #pragma unroll
@@ -662,7 +730,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
         for (int n = 0; n < ZT; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e)
-            sDecay[(m * 16 + lr + (e >> 1) * 8) * DP + warp * (DP / 8) + n * 8 + lc + (e & 1)] = expf(g[m][n][e]);
+            sDecay[(m * 16 + lr + (e >> 1) * 8) * DP + warp * (DP / 8) + n * 8 + lc + (e & 1)] = exp2f(g[m][n][e]);
       __syncthreads();
       if (owner) {
         for (int t = 0; t < rows; ++t) {
@@ -718,6 +786,8 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
           }
         }
       }
+      __syncthreads();
+      load_gate();
     }
     if (kStateOnly) continue;
 
@@ -751,42 +821,47 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
           if ((lane & 3) == 0) sRow[(m * 16 + lr + half * 8) * 8 + warp] = sq;
         }
     }
+    cp_wait_all();
     __syncthreads();
     if (owner) {
+      // Dead rows have zero outputs and gates.
 #pragma unroll
       for (int m = 0; m < 4; ++m)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int r = m * 16 + lr + half * 8;
-          if (t0 + r >= t_hi) continue;
-          float total = 0.f;
-#pragma unroll
-          for (int w = 0; w < kWarpsV; ++w) total += sRow[r * 8 + w];
-          const float inv = rsqrtf(total / a.vdim + a.eps);
-          const int64_t tok = static_cast<int64_t>(b) * a.T + t0 + r;
-          bf16* out = static_cast<bf16*>(a.out) + tok * a.out_ld + h * a.vdim;
-          const bf16* gate = base + static_cast<int64_t>(t0 + r) * a.ld + a.g_off + h * a.vdim;
+          const float4 s0 = *reinterpret_cast<const float4*>(sRow + r * 8);
+          float total = s0.x + s0.y + s0.z + s0.w;
+          if (kWarpsV > 4) {
+            const float4 s1 = *reinterpret_cast<const float4*>(sRow + r * 8 + 4);
+            total += s1.x + s1.y + s1.z + s1.w;
+          }
+          const float inv = rsqrtf(total * inv_vdim + a.eps);
 #pragma unroll
           for (int n = 0; n < MV * 2; ++n) {
-            const int v = v0 + n * 8 + lc;
-            float y[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-              y[e] = 0.f;
-              if (r < rows && v + e < vcols) {
-                const float x = __bfloat162float(gate[v + e]);
-                y[e] = O[m][n][half * 2 + e] * inv * a.norm_w[v + e] * (x / (1.f + __expf(-x)));
-              }
-            }
-            if (vec && v < vcols) {
-              *reinterpret_cast<uint32_t*>(out + v) = pack2(y[0], y[1]);
-            } else {
-#pragma unroll
-              for (int e = 0; e < 2; ++e)
-                if (v + e < vcols) out[v + e] = __float2bfloat16(y[e]);
-            }
+            uint32_t* p = reinterpret_cast<uint32_t*>(sQ + r * L::kVP + v0 + n * 8 + lc);
+            const float2 x = unpack2(*p);
+            *p = pack2(O[m][n][half * 2] * inv * nw[n][0] * silu_fast(x.x),
+                       O[m][n][half * 2 + 1] * inv * nw[n][1] * silu_fast(x.y));
           }
         }
+    }
+    __syncthreads();
+    const int n_out = min(kGcTok, t_hi - t0);
+    bf16* out = static_cast<bf16*>(a.out) + (static_cast<int64_t>(b) * a.T + t0) * a.out_ld + h * a.vdim;
+    if (vec) {
+      const int c = (tid % (VS / 8)) * 8;
+      bf16* p = out + (tid / (VS / 8)) * a.out_ld + c;
+#pragma unroll
+      for (int r = tid / (VS / 8); r < kGcTok; r += kGcThreads / (VS / 8)) {
+        if (r < n_out && c < vcols) *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(sQ + r * L::kVP + c);
+        p += kGcThreads / (VS / 8) * a.out_ld;
+      }
+    } else {
+      for (int i = tid; i < n_out * vcols; i += kGcThreads) {
+        const int r = i / vcols, c = i % vcols;
+        out[r * a.out_ld + c] = sQ[r * L::kVP + c];
+      }
     }
   }
 
@@ -823,7 +898,7 @@ __global__ void gla_segment_kernel(GlaArgs a) {
     float* p = a.seg_state + (bh * a.segments + g) * n + i;
     const float add = *p;
     *p = s;
-    s = s * expf(a.seg_decay[(bh * a.segments + g) * a.dim + c]) + add;
+    s = s * exp2f(a.seg_decay[(bh * a.segments + g) * a.dim + c]) + add;
   }
 }
 

@@ -32,7 +32,7 @@ struct WindowArgs {
   void* out;             // [B, T, out_ld]
   const int* start;
   const int* live;
-  float* part;           // decode splits: [B, H, splits, vdim + 2]
+  float* part;           // decode splits: [B, H, splits, vdim + 2 rounded up to 4]
   int* tickets;          // [B * CTA groups], zero on entry and on exit
   int64_t ld, out_ld;
   int B, T, heads, kv_heads, dim, vdim, slots, window;
@@ -55,55 +55,53 @@ __device__ __forceinline__ float head_slope(const WindowArgs& a, int h) {
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
-// 16 bytes of a row starting at element `c` of `n`; elements at or beyond n are zero.
-template <bool kAligned>
-__device__ __forceinline__ void load_chunk(const __nv_bfloat16* p, int c, int n, float* f) {
+// 16 bytes of a row starting at element `c` of `n`, raw; elements at or beyond n are zero.
+template <typename T, bool kAligned>
+__device__ __forceinline__ uint4 load_raw(const T* p, int c, int n) {
+  uint4 u = make_uint4(0, 0, 0, 0);
   if (kAligned) {
-    uint4 u = make_uint4(0, 0, 0, 0);
     if (c < n) u = *reinterpret_cast<const uint4*>(p + c);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 t = __bfloat1622float2(h[i]);
-      f[2 * i] = t.x, f[2 * i + 1] = t.y;
-    }
   } else {
+    T* e = reinterpret_cast<T*>(&u);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) f[i] = c + i < n ? __bfloat162float(p[c + i]) : 0.f;
+    for (int i = 0; i < static_cast<int>(16 / sizeof(T)); ++i)
+      if (c + i < n) e[i] = p[c + i];
+  }
+  return u;
+}
+template <typename T>
+__device__ __forceinline__ void expand(const uint4& u, float* f);
+template <>
+__device__ __forceinline__ void expand<__nv_bfloat16>(const uint4& u, float* f) {
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 t = __bfloat1622float2(h[i]);
+    f[2 * i] = t.x, f[2 * i + 1] = t.y;
   }
 }
-template <bool kAligned>
-__device__ __forceinline__ void load_chunk(const float* p, int c, int n, float* f) {
-  if (kAligned) {
-    float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < n) u = *reinterpret_cast<const float4*>(p + c);
-    f[0] = u.x, f[1] = u.y, f[2] = u.z, f[3] = u.w;
-  } else {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) f[i] = c + i < n ? p[c + i] : 0.f;
-  }
-}
-// A lane's share of a head row: E elements in 16-byte chunks, chunk i at (lane8 + 8 i) * chunk size.
-template <typename T, int E, bool kAligned>
-__device__ __forceinline__ void load_share(const T* row, int lane8, int n, float (&f)[E]) {
-  constexpr int VEC = 16 / sizeof(T);
-#pragma unroll
-  for (int i = 0; i < E / VEC; ++i) load_chunk<kAligned>(row, (lane8 + 8 * i) * VEC, n, f + i * VEC);
+template <>
+__device__ __forceinline__ void expand<float>(const uint4& u, float* f) {
+  f[0] = __uint_as_float(u.x), f[1] = __uint_as_float(u.y), f[2] = __uint_as_float(u.z), f[3] = __uint_as_float(u.w);
 }
 
-constexpr int kWdThreads = 128;
+constexpr int kWdThreads = 256, kWdWarps = kWdThreads / 32, kMaxSplits = 64;
 
 }  // namespace
 
-// Eight lanes share a key; a warp covers four keys, the CTA sixteen.  GT query heads of one KV head.
-template <typename T, int GT, int EK, int EV, bool kAligned>
-__global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WindowArgs a) {
+// LPK lanes share a key, NC 16-byte chunks of the head row each (chunk i of lane l at (l + LPK i) * 16
+// bytes); a warp covers 32 / LPK keys per step and keeps U steps' loads in flight.  GT query heads of one KV
+// head per CTA.
+template <typename T, int GT, int LPK, int NC, int U, bool kAligned>
+__global__ void __launch_bounds__(kWdThreads, 2) window_decode_kernel(WindowArgs a) {
   constexpr int VEC = 16 / sizeof(T);
-  constexpr int U = EK <= 8 ? 4 : EK <= 16 ? (GT == 1 ? 4 : 2) : 1;  // keys per lane group in flight
+  constexpr int E = NC * VEC;                // elements per lane
+  constexpr int KPW = 32 / LPK;              // keys per warp and step
+  constexpr int STEP = KPW * kWdWarps;
   const int split = blockIdx.x, b = blockIdx.z;
   const int per_kv = a.heads / a.kv_heads, groups = per_kv / GT;
   const int kvh = blockIdx.y / groups, qh0 = kvh * per_kv + (blockIdx.y % groups) * GT;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, slot4 = lane >> 3, lane8 = lane & 7;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, slot = lane / LPK, lk = lane % LPK;
   const int pos = a.start[b];
   T* out = static_cast<T*>(a.out) + static_cast<int64_t>(b) * a.out_ld;
   if (pos < 0 || (a.live != nullptr && a.live[b] <= 0)) {  // row not in this step
@@ -112,135 +110,166 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WindowArgs a)
     return;
   }
   const T* row = static_cast<const T*>(a.proj) + static_cast<int64_t>(b) * a.ld;
-  T* k_ring = static_cast<T*>(a.k_ring) + static_cast<int64_t>(b) * a.slots * a.kv_heads * a.dim;
-  T* v_ring = static_cast<T*>(a.v_ring) + static_cast<int64_t>(b) * a.slots * a.kv_heads * a.vdim;
+  T* k_ring = static_cast<T*>(a.k_ring) + (static_cast<int64_t>(b) * a.slots * a.kv_heads + kvh) * a.dim;
+  T* v_ring = static_cast<T*>(a.v_ring) + (static_cast<int64_t>(b) * a.slots * a.kv_heads + kvh) * a.vdim;
+  const int64_t k_pitch = static_cast<int64_t>(a.kv_heads) * a.dim, v_pitch = static_cast<int64_t>(a.kv_heads) * a.vdim;
   const T* k_new = row + a.k_off + kvh * a.dim;
   const T* v_new = row + a.v_off + kvh * a.vdim;
-  if (split == 0 && blockIdx.y % groups == 0) {
-    // The slot being written holds the key that has just left the window: nobody reads it.
-    const int s = pos % a.slots;
-    T* kd = k_ring + (static_cast<int64_t>(s) * a.kv_heads + kvh) * a.dim;
-    T* vd = v_ring + (static_cast<int64_t>(s) * a.kv_heads + kvh) * a.vdim;
-    for (int c = threadIdx.x; c < a.dim; c += kWdThreads) kd[c] = k_new[c];
-    for (int c = threadIdx.x; c < a.vdim; c += kWdThreads) vd[c] = v_new[c];
-  }
   const int lo = max(0, pos + 1 - min(a.window, a.slots));
   const int count = pos - lo + 1;
   const int per = (count + a.splits - 1) / a.splits;
   const int j_lo = lo + split * per, j_hi = min(pos + 1, j_lo + per);
 
-  float q[GT][EK], acc[GT][EV], m[GT], l[GT], slope[GT];
+  float q[GT][E], acc[GT][E], m[GT], l[GT], slope[GT];
   const float qs = query_scale(a, pos) * 1.4426950408889634f;
 #pragma unroll
   for (int g = 0; g < GT; ++g) {
-    load_share<T, EK, kAligned>(row + a.q_off + (qh0 + g) * a.dim, lane8, a.dim, q[g]);
 #pragma unroll
-    for (int i = 0; i < EK; ++i) q[g][i] *= qs;
+    for (int i = 0; i < NC; ++i)
+      expand<T>(load_raw<T, kAligned>(row + a.q_off + (qh0 + g) * a.dim, (lk + LPK * i) * VEC, a.dim), q[g] + i * VEC);
 #pragma unroll
-    for (int i = 0; i < EV; ++i) acc[g][i] = 0.f;
+    for (int i = 0; i < E; ++i) q[g][i] *= qs, acc[g][i] = 0.f;
     m[g] = -INFINITY, l[g] = 0.f;
     slope[g] = head_slope(a, qh0 + g) * 1.4426950408889634f;
   }
-  for (int j0 = j_lo + warp * 4 + slot4; j0 - slot4 < j_hi; j0 += 16 * U) {
-    float kf[U][EK], vf[U][EV];
+  // Ring slot of a key, kept by addition: a step moves every lane group by STEP keys.
+  int j = j_lo + warp * KPW + slot;
+  int at = j % a.slots;
+  const int step_slots = STEP % a.slots;
+  for (; j - slot < j_hi;) {
+    uint4 kr[U][NC], vr[U][NC];
+    bool ok[U];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      const int j = j0 + 16 * u;
-      if (j < j_hi) {
-        const int s = j % a.slots;
-        const T* kp = j == pos ? k_new : k_ring + (static_cast<int64_t>(s) * a.kv_heads + kvh) * a.dim;
-        const T* vp = j == pos ? v_new : v_ring + (static_cast<int64_t>(s) * a.kv_heads + kvh) * a.vdim;
-        load_share<T, EK, kAligned>(kp, lane8, a.dim, kf[u]);
-        load_share<T, EV, kAligned>(vp, lane8, a.vdim, vf[u]);
-      } else {
+      const int ju = j + STEP * u;
+      ok[u] = ju < j_hi;
+      const T* kp = ju == pos ? k_new : k_ring + at * k_pitch;
+      const T* vp = ju == pos ? v_new : v_ring + at * v_pitch;
 #pragma unroll
-        for (int i = 0; i < EK; ++i) kf[u][i] = 0.f;
+      for (int i = 0; i < NC; ++i) {
+        kr[u][i] = vr[u][i] = make_uint4(0, 0, 0, 0);
+        if (ok[u]) {
+          kr[u][i] = load_raw<T, kAligned>(kp, (lk + LPK * i) * VEC, a.dim);
+          vr[u][i] = load_raw<T, kAligned>(vp, (lk + LPK * i) * VEC, a.vdim);
+        }
+      }
+      at += step_slots;
+      if (at >= a.slots) at -= a.slots;
+    }
+    float s[GT][U];
 #pragma unroll
-        for (int i = 0; i < EV; ++i) vf[u][i] = 0.f;
+    for (int u = 0; u < U; ++u) {
+      float kf[E];
+#pragma unroll
+      for (int i = 0; i < NC; ++i) expand<T>(kr[u][i], kf + i * VEC);
+#pragma unroll
+      for (int g = 0; g < GT; ++g) {
+        float d = 0.f;
+#pragma unroll
+        for (int i = 0; i < E; ++i) d += q[g][i] * kf[i];
+        s[g][u] = d;
       }
     }
 #pragma unroll
+    for (int off = 1; off < LPK; off <<= 1)
+#pragma unroll
+      for (int g = 0; g < GT; ++g)
+#pragma unroll
+        for (int u = 0; u < U; ++u) s[g][u] += __shfl_xor_sync(0xffffffffu, s[g][u], off);
+#pragma unroll
     for (int g = 0; g < GT; ++g) {
-      float s[U], mx = m[g];
+      float mx = m[g];
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        const int j = j0 + 16 * u;
-        float d = 0.f;
-#pragma unroll
-        for (int i = 0; i < EK; ++i) d += q[g][i] * kf[u][i];
-        d += __shfl_xor_sync(0xffffffffu, d, 1);
-        d += __shfl_xor_sync(0xffffffffu, d, 2);
-        d += __shfl_xor_sync(0xffffffffu, d, 4);
-        s[u] = j < j_hi ? d - slope[g] * static_cast<float>(pos - j) : -INFINITY;
-        mx = fmaxf(mx, s[u]);
+        s[g][u] = ok[u] ? s[g][u] - slope[g] * static_cast<float>(pos - j - STEP * u) : -INFINITY;
+        mx = fmaxf(mx, s[g][u]);
       }
       const bool none = mx == -INFINITY;  // no key for this lane group yet
       const float corr = none ? 1.f : exp2f(m[g] - mx);
       l[g] *= corr;
 #pragma unroll
-      for (int i = 0; i < EV; ++i) acc[g][i] *= corr;
+      for (int i = 0; i < E; ++i) acc[g][i] *= corr;
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        const float p = none ? 0.f : exp2f(s[u] - mx);
-        l[g] += p;
-#pragma unroll
-        for (int i = 0; i < EV; ++i) acc[g][i] += p * vf[u][i];
+        s[g][u] = none ? 0.f : exp2f(s[g][u] - mx);
+        l[g] += s[g][u];
       }
       m[g] = mx;
     }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      float vf[E];
+#pragma unroll
+      for (int i = 0; i < NC; ++i) expand<T>(vr[u][i], vf + i * VEC);
+#pragma unroll
+      for (int g = 0; g < GT; ++g)
+#pragma unroll
+        for (int i = 0; i < E; ++i) acc[g][i] += s[g][u] * vf[i];
+    }
+    j += STEP * U;
+  }
+  if (split == 0 && blockIdx.y % groups == 0) {
+    // The slot being written holds the key that has just left the window: nobody reads it.
+    const int64_t s = pos % a.slots;
+    for (int c = threadIdx.x; c < a.dim; c += kWdThreads) k_ring[s * k_pitch + c] = k_new[c];
+    for (int c = threadIdx.x; c < a.vdim; c += kWdThreads) v_ring[s * v_pitch + c] = v_new[c];
   }
 
-  // Four lane groups of a warp, then four warps.
-  __shared__ float s_m[4][GT], s_l[4][GT], s_acc[4][GT][8 * EV];
+  // Lane groups of a warp, then the warps.
+  __shared__ float s_m[kWdWarps][GT], s_l[kWdWarps][GT], s_acc[kWdWarps][GT][LPK * E];
+  __shared__ float s_c[GT][kWdWarps];
   __shared__ int s_last;
 #pragma unroll
   for (int g = 0; g < GT; ++g) {
 #pragma unroll
-    for (int off = 8; off <= 16; off <<= 1) {
+    for (int off = LPK; off < 32; off <<= 1) {
       const float mo = __shfl_xor_sync(0xffffffffu, m[g], off), lo_ = __shfl_xor_sync(0xffffffffu, l[g], off);
       const float mn = fmaxf(m[g], mo);
       const float cs = mn == -INFINITY ? 1.f : exp2f(m[g] - mn), co = mn == -INFINITY ? 1.f : exp2f(mo - mn);
       l[g] = l[g] * cs + lo_ * co;
 #pragma unroll
-      for (int i = 0; i < EV; ++i)
+      for (int i = 0; i < E; ++i)
         acc[g][i] = acc[g][i] * cs + __shfl_xor_sync(0xffffffffu, acc[g][i], off) * co;
       m[g] = mn;
     }
-    if (slot4 == 0) {
+    if (slot == 0) {
 #pragma unroll
-      for (int i = 0; i < EV; ++i) s_acc[warp][g][(lane8 + 8 * (i / VEC)) * VEC + i % VEC] = acc[g][i];
-      if (lane8 == 0) s_m[warp][g] = m[g], s_l[warp][g] = l[g];
+      for (int i = 0; i < E; ++i) s_acc[warp][g][(lk + LPK * (i / VEC)) * VEC + i % VEC] = acc[g][i];
+      if (lk == 0) s_m[warp][g] = m[g], s_l[warp][g] = l[g];
     }
   }
   __syncthreads();
-  const int pitch = a.vdim + 2;
-#pragma unroll
-  for (int g = 0; g < GT; ++g) {
-    float mm = -INFINITY;
-#pragma unroll
-    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, s_m[w][g]);
-    float c[4], ll = 0.f;
-#pragma unroll
-    for (int w = 0; w < 4; ++w) {
-      c[w] = mm == -INFINITY ? 0.f : exp2f(s_m[w][g] - mm);
-      ll += s_l[w][g] * c[w];
+  const int pitch = (a.vdim + 5) & ~3;  // outputs, then maximum and sum
+  float* part = a.part + (static_cast<int64_t>(b) * a.heads + qh0) * a.splits * pitch;  // [GT][splits][pitch]
+  if (threadIdx.x < GT) {
+    const int g = threadIdx.x;
+    float mm = -INFINITY, ll = 0.f;
+    for (int w = 0; w < kWdWarps; ++w) mm = fmaxf(mm, s_m[w][g]);
+    for (int w = 0; w < kWdWarps; ++w) {
+      const float c = mm == -INFINITY ? 0.f : exp2f(s_m[w][g] - mm);
+      ll += s_l[w][g] * c;
+      s_c[g][w] = c;
     }
-    float* part = a.splits == 1 ? nullptr
-                                : a.part + ((static_cast<int64_t>(b) * a.heads + qh0 + g) * a.splits + split) * pitch;
-    for (int d = threadIdx.x; d < a.vdim; d += kWdThreads) {
-      float o = 0.f;
-#pragma unroll
-      for (int w = 0; w < 4; ++w) o += s_acc[w][g][d] * c[w];
-      if (a.splits == 1) {
-        o /= ll;
-        const int col = (qh0 + g) * a.vdim + d;
-        if (a.g_off >= 0) o *= sigmoid_f(to_f(row[a.g_off + col]));
-        out[col] = T(o);
-      } else {
-        part[d] = o;
-      }
+    if (a.splits == 1) {
+      for (int w = 0; w < kWdWarps; ++w) s_c[g][w] /= ll;
+    } else {
+      float* mine = part + (g * a.splits + split) * pitch + a.vdim;
+      mine[0] = mm, mine[1] = ll;
     }
-    if (a.splits > 1 && threadIdx.x == 0) part[a.vdim] = mm, part[a.vdim + 1] = ll;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < GT * a.vdim; i += kWdThreads) {
+    const int g = i / a.vdim, d = i % a.vdim;
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < kWdWarps; ++w) o += s_acc[w][g][d] * s_c[g][w];
+    if (a.splits == 1) {
+      const int col = qh0 * a.vdim + i;
+      if (a.g_off >= 0) o *= sigmoid_f(to_f(row[a.g_off + col]));
+      out[col] = T(o);
+    } else {
+      part[(g * a.splits + split) * pitch + d] = o;
+    }
   }
   if (a.splits == 1) return;
   // The last CTA of this (sequence, head group) merges the splits.
@@ -252,21 +281,52 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WindowArgs a)
   if (!s_last) return;
   __threadfence();
   if (threadIdx.x == 0) *ticket = 0;
-#pragma unroll 1
-  for (int g = 0; g < GT; ++g) {
-    const float* base = a.part + (static_cast<int64_t>(b) * a.heads + qh0 + g) * a.splits * pitch;
-    float mm = -INFINITY;
-    for (int s = 0; s < a.splits; ++s) mm = fmaxf(mm, __ldcg(base + s * pitch + a.vdim));
-    float ll = 0.f;
-    for (int s = 0; s < a.splits; ++s)
-      ll += __ldcg(base + s * pitch + a.vdim + 1) * exp2f(__ldcg(base + s * pitch + a.vdim) - mm);
-    for (int d = threadIdx.x; d < a.vdim; d += kWdThreads) {
-      float o = 0.f;
-      for (int s = 0; s < a.splits; ++s) o += __ldcg(base + s * pitch + d) * exp2f(__ldcg(base + s * pitch + a.vdim) - mm);
-      o /= ll;
+  // Weight of every split: one warp per head.
+  __shared__ float s_w[GT][kMaxSplits];
+  if (warp < GT) {
+    const int g = warp;
+    float mv[kMaxSplits / 32], lv[kMaxSplits / 32], mm = -INFINITY, ll = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) {
+      const int s = lane + 32 * i;
+      const float* p = part + (g * a.splits + s) * pitch + a.vdim;
+      mv[i] = s < a.splits ? __ldcg(p) : -INFINITY;
+      lv[i] = s < a.splits ? __ldcg(p + 1) : 0.f;
+      mm = fmaxf(mm, mv[i]);
+    }
+    for (int off = 16; off > 0; off >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, off));
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) mv[i] = exp2f(mv[i] - mm), ll += lv[i] * mv[i];
+    for (int off = 16; off > 0; off >>= 1) ll += __shfl_xor_sync(0xffffffffu, ll, off);
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) s_w[g][lane + 32 * i] = mv[i] / ll;
+  }
+  __syncthreads();
+  auto finish = [&](int col, float o) {
+    if (a.g_off >= 0) o *= sigmoid_f(to_f(row[a.g_off + col]));
+    out[col] = T(o);
+  };
+  if (a.vdim % 4 == 0) {
+    for (int i = threadIdx.x; i < GT * (a.vdim / 4); i += kWdThreads) {
+      const int g = i / (a.vdim / 4), d = (i % (a.vdim / 4)) * 4;
+      const float* p = part + g * a.splits * pitch + d;
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+      for (int s = 0; s < a.splits; ++s) {
+        const float4 x = __ldcg(reinterpret_cast<const float4*>(p + s * pitch));
+        const float w = s_w[g][s];
+        o.x += x.x * w, o.y += x.y * w, o.z += x.z * w, o.w += x.w * w;
+      }
       const int col = (qh0 + g) * a.vdim + d;
-      if (a.g_off >= 0) o *= sigmoid_f(to_f(row[a.g_off + col]));
-      out[col] = T(o);
+      finish(col, o.x), finish(col + 1, o.y), finish(col + 2, o.z), finish(col + 3, o.w);
+    }
+  } else {
+    for (int i = threadIdx.x; i < GT * a.vdim; i += kWdThreads) {
+      const int g = i / a.vdim;
+      const float* p = part + g * a.splits * pitch + i % a.vdim;
+      float o = 0.f;
+      for (int s = 0; s < a.splits; ++s) o += __ldcg(p + s * pitch) * s_w[g][s];
+      finish(qh0 * a.vdim + i, o);
     }
   }
 }
@@ -377,19 +437,30 @@ __global__ void __launch_bounds__(kWaThreads) window_attn_kernel(WindowArgs a) {
   }
 }
 
-template <typename T>
-__global__ void window_append_kernel(WindowArgs a) {
+// V: 16-byte vectors (row sizes, pitches and offsets permitting) or single elements.
+template <typename V, typename T>
+__global__ void __launch_bounds__(128) window_append_kernel(WindowArgs a) {
+  constexpr int N = sizeof(V) / sizeof(T);
   const int b = blockIdx.y;
   const int start = a.start != nullptr ? a.start[b] : 0;
   const int live = a.live != nullptr ? min(a.live[b], a.T) : a.T;
-  const int t = live - 1 - static_cast<int>(blockIdx.x);
-  if (t < 0 || start < 0) return;
-  const T* row = static_cast<const T*>(a.proj) + (static_cast<int64_t>(b) * a.T + t) * a.ld;
-  const int64_t slot = static_cast<int64_t>(b) * a.slots + (start + t) % a.slots;
-  T* kd = static_cast<T*>(a.k_ring) + slot * a.kv_heads * a.dim;
-  T* vd = static_cast<T*>(a.v_ring) + slot * a.kv_heads * a.vdim;
-  for (int c = threadIdx.x; c < a.kv_heads * a.dim; c += blockDim.x) kd[c] = row[a.k_off + c];
-  for (int c = threadIdx.x; c < a.kv_heads * a.vdim; c += blockDim.x) vd[c] = row[a.v_off + c];
+  const int kc = a.kv_heads * a.dim / N, vc = a.kv_heads * a.vdim / N;
+  for (int back = blockIdx.x; back < a.slots; back += gridDim.x) {
+    const int t = live - 1 - back;
+    if (t < 0 || start < 0) return;
+    const T* row = static_cast<const T*>(a.proj) + (static_cast<int64_t>(b) * a.T + t) * a.ld;
+    const int64_t slot = static_cast<int64_t>(b) * a.slots + (start + t) % a.slots;
+    const V* ks = reinterpret_cast<const V*>(row + a.k_off);
+    const V* vs = reinterpret_cast<const V*>(row + a.v_off);
+    V* kd = reinterpret_cast<V*>(static_cast<T*>(a.k_ring)) + slot * kc;
+    V* vd = reinterpret_cast<V*>(static_cast<T*>(a.v_ring)) + slot * vc;
+    for (int c = threadIdx.x; c < kc + vc; c += blockDim.x) {
+      if (c < kc)
+        kd[c] = ks[c];
+      else
+        vd[c - kc] = vs[c - kc];
+    }
+  }
 }
 
 template <typename T>
@@ -414,23 +485,25 @@ static int query_heads_per_cta(int heads, int kv_heads) {
   return per_kv % 4 == 0 ? 4 : per_kv % 2 == 0 ? 2 : 1;
 }
 
-template <typename T, int GT, int EK, int EV>
+template <typename T, int GT, int LPK, int NC, int U>
 static int launch_decode(const WindowArgs& a, bool aligned, cudaStream_t stream) {
   const dim3 grid(a.splits, a.heads / GT, a.B);
   if (aligned)
-    window_decode_kernel<T, GT, EK, EV, true><<<grid, kWdThreads, 0, stream>>>(a);
+    window_decode_kernel<T, GT, LPK, NC, U, true><<<grid, kWdThreads, 0, stream>>>(a);
   else
-    window_decode_kernel<T, GT, EK, EV, false><<<grid, kWdThreads, 0, stream>>>(a);
+    window_decode_kernel<T, GT, LPK, NC, U, false><<<grid, kWdThreads, 0, stream>>>(a);
   return cudaGetLastError() == cudaSuccess ? zero_tail<T>(a, stream) : -4;
 }
 
+// Eight bf16 (or two times four fp32) elements per lane; 512-element heads take twice that.
 template <typename T, int GT>
 static int dispatch_decode(const WindowArgs& a, bool aligned, cudaStream_t stream) {
-  const int e = (a.dim > a.vdim ? a.dim : a.vdim);
-  if (e <= 64) return launch_decode<T, GT, 8, 8>(a, aligned, stream);
-  if (e <= 128) return launch_decode<T, GT, 16, 16>(a, aligned, stream);
-  if (e <= 256) return launch_decode<T, (GT > 2 ? 2 : GT), 32, 32>(a, aligned, stream);
-  return launch_decode<T, 1, 64, 64>(a, aligned, stream);
+  constexpr int N = sizeof(T) / 2, U = (GT == 4 ? 2 : 4) / N;
+  const int e = a.dim > a.vdim ? a.dim : a.vdim;
+  if (e <= 64) return launch_decode<T, GT, 8, N, U>(a, aligned, stream);
+  if (e <= 128) return launch_decode<T, GT, 16, N, U>(a, aligned, stream);
+  if (e <= 256) return launch_decode<T, GT, 32, N, U>(a, aligned, stream);
+  return launch_decode<T, (GT > 2 ? 2 : GT), 32, 2 * N, 1>(a, aligned, stream);
 }
 
 template <typename T>
@@ -461,6 +534,19 @@ static int window_attn(const WindowArgs& a, cudaStream_t stream) {
   return cudaGetLastError() == cudaSuccess ? zero_tail<T>(a, stream) : -4;
 }
 
+template <typename T>
+static int window_append(const WindowArgs& a, cudaStream_t stream) {
+  constexpr int VEC = 16 / sizeof(T);
+  const int tokens = a.T < a.slots ? a.T : a.slots;
+  const dim3 grid(tokens < 1024 ? tokens : 1024, a.B);
+  auto ok = [](int64_t x) { return x % VEC == 0; };
+  if (ok(a.ld) && ok(a.k_off) && ok(a.v_off) && ok(a.kv_heads * a.dim) && ok(a.kv_heads * a.vdim))
+    window_append_kernel<uint4, T><<<grid, 128, 0, stream>>>(a);
+  else
+    window_append_kernel<T, T><<<grid, 128, 0, stream>>>(a);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 static bool bad(const WindowArgs& a) {
   return a.B <= 0 || a.T <= 0 || a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 ||
          a.vdim <= 0 || a.dim > 512 || a.vdim > 512 || a.slots <= 0 || a.window <= 0 || a.every <= 0 ||
@@ -472,16 +558,14 @@ static bool bad(const WindowArgs& a) {
 // CTAs of one KV split of the decode kernel (the caller sizes `splits` and `tickets` by it).
 extern "C" int axb_window_decode_ctas(int B, int heads, int kv_heads, int dim, int vdim) {
   int gt = axb::query_heads_per_cta(heads, kv_heads);
-  const int e = dim > vdim ? dim : vdim;
-  if (e > 128 && gt > 2) gt = 2;
-  if (e > 256) gt = 1;
+  if ((dim > vdim ? dim : vdim) > 256 && gt > 2) gt = 2;
   return B * (heads / gt);
 }
 
 // One new token per sequence (T == 1, `start` required).
 extern "C" int axb_window_decode(const axb::WindowArgs* args, cudaStream_t stream) {
   const axb::WindowArgs& a = *args;
-  if (axb::bad(a) || a.T != 1 || a.start == nullptr || a.splits < 1) return -10;
+  if (axb::bad(a) || a.T != 1 || a.start == nullptr || a.splits < 1 || a.splits > axb::kMaxSplits) return -10;
   if (a.splits > 1 && (a.part == nullptr || a.tickets == nullptr)) return -11;
   return a.act_bf16 ? axb::window_decode<__nv_bfloat16>(a, stream) : axb::window_decode<float>(a, stream);
 }
@@ -497,10 +581,5 @@ extern "C" int axb_window_attn(const axb::WindowArgs* args, cudaStream_t stream)
 extern "C" int axb_window_append(const axb::WindowArgs* args, cudaStream_t stream) {
   const axb::WindowArgs& a = *args;
   if (axb::bad(a)) return -10;
-  const dim3 grid(a.T < a.slots ? a.T : a.slots, a.B);
-  if (a.act_bf16)
-    axb::window_append_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(a);
-  else
-    axb::window_append_kernel<float><<<grid, 128, 0, stream>>>(a);
-  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  return a.act_bf16 ? axb::window_append<__nv_bfloat16>(a, stream) : axb::window_append<float>(a, stream);
 }

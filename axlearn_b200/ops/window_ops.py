@@ -192,9 +192,9 @@ def _ticket_buffer(device: torch.device, n: int) -> Tensor:
 
 
 def decode_splits(ctas: int, span: int, sms: int = 148) -> int:
-    """KV splits of a decoding step: about four CTAs per SM, at least 64 keys each."""
-    want = max(1, (4 * sms) // max(1, ctas))
-    return max(1, min(want, span // 64 if span >= 64 else 1, 64))
+    """KV splits of a decoding step: one wave of two CTAs per SM, at least 64 keys each."""
+    want = max(1, (2 * sms) // max(1, ctas))
+    return max(1, min(want, span // 64, 64))
 
 
 def flash_supported(proj: Tensor, spec: WindowSpec, cols: WindowColumns) -> bool:
@@ -239,7 +239,7 @@ def _cuda_window_attention(proj, spec, cols, *, start, live, cache):
         a.splits = decode_splits(ctas, min(spec.window, a.slots))
         part = None
         if a.splits > 1:
-            part = torch.empty(b * spec.heads * a.splits * (spec.vdim + 2), dtype=torch.float32, device=proj.device)
+            part = torch.empty(b * spec.heads * a.splits * padded(spec.vdim + 2, 4), dtype=torch.float32, device=proj.device)
             a.part, a.tickets = part.data_ptr(), _ticket_buffer(proj.device, ctas).data_ptr()
         check(lib.axb_window_decode(ctypes.byref(a), stream), "axb_window_decode")
         return out, cache
