@@ -399,7 +399,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
   const bool vec_a1 = vec && !((a.a1_off | a.rank) & 7);
   const bool owner = warp < kWarpsV;
   const int v0 = warp * 16 * MV;  // first value column of this warp in the slice
-  const float inv_vdim = 1.f / a.vdim;
+  const float mean_scale = a.q_scale * a.q_scale / a.vdim;  // outputs are scaled by q_scale at the end
   float nw[MV * 2][2];
 #pragma unroll
   for (int n = 0; n < MV * 2; ++n)
@@ -591,7 +591,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
             if (!kStateOnly) {
               uint32_t* pq = reinterpret_cast<uint32_t*>(sQ + r * L::kQP + c);
               const float2 q = unpack2(*pq);
-              *pq = pack2(q.x * a.q_scale * ex2(g0), q.y * a.q_scale * ex2(g1));
+              *pq = pack2(q.x * ex2(g0), q.y * ex2(g1));
             }
             uint32_t* pk = reinterpret_cast<uint32_t*>(sK + r * L::kQP + c);
             const float2 k = unpack2(*pk);
@@ -768,7 +768,6 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
                 float x = o[mv][u];
                 x += __shfl_xor_sync(0xffffffffu, x, 1);
                 x += __shfl_xor_sync(0xffffffffu, x, 2);
-                x *= a.q_scale;
                 // Lane (lr, *) now holds token t, column lr + 8 u; an O fragment wants row t at lanes with
                 // lr == t % 8, columns 2 (lane & 3), + 1.
                 const float y0 = __shfl_sync(0xffffffffu, x, lc * 4), y1 = __shfl_sync(0xffffffffu, x, (lc + 1) * 4);
@@ -802,7 +801,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
             for (int e = 0; e < 4; ++e) {
               const int r = m * 16 + lr + (e >> 1) * 8, v = v0 + n * 8 + lc + (e & 1);
               if (r < rows && v < vcols)
-                a.o_raw[((static_cast<int64_t>(b) * a.T + t0 + r) * a.heads + h) * a.vdim + d0 + v] = O[m][n][e];
+                a.o_raw[((static_cast<int64_t>(b) * a.T + t0 + r) * a.heads + h) * a.vdim + d0 + v] = O[m][n][e] * a.q_scale;
             }
       }
       continue;
@@ -836,7 +835,7 @@ __global__ void __launch_bounds__(kGcThreads, 2) gla_chunk_kernel(GlaArgs a) {
             const float4 s1 = *reinterpret_cast<const float4*>(sRow + r * 8 + 4);
             total += s1.x + s1.y + s1.z + s1.w;
           }
-          const float inv = rsqrtf(total * inv_vdim + a.eps);
+          const float inv = a.q_scale * rsqrtf(total * mean_scale + a.eps);
 #pragma unroll
           for (int n = 0; n < MV * 2; ++n) {
             uint32_t* p = reinterpret_cast<uint32_t*>(sQ + r * L::kVP + v0 + n * 8 + lc);
