@@ -202,7 +202,7 @@ class GatedLinearAttention(BaseSequenceMixer):
 
 
 class ParallelMixer(BaseLayer):
-    """Two mixers side by side on one input: the mean of their outputs, each RMS-normed over the model
+    """Two mixers that share one input: the mean of their outputs, each RMS-normed over the model
     width with a plain weight.  One product computes both mixers' projections.
 
     ``forward`` returns the two raw outputs as a ``NormedPair``; the norms and the mean are part of the

@@ -37,8 +37,27 @@ def _nvcc() -> str:
     return "nvcc"
 
 
-def sources() -> list[str]:
-    return sorted(os.path.join(HERE, f) for f in os.listdir(HERE) if f.endswith(".cu"))
+def sources(only=None) -> list[str]:
+    """Paths of all ``.cu`` files, or of those named in ``only``."""
+    names = sorted(f for f in os.listdir(HERE) if f.endswith(".cu"))
+    if only is not None:
+        missing = set(only) - set(names)
+        if missing:
+            raise ValueError(f"no such sources: {sorted(missing)}")
+        names = [f for f in names if f in set(only)]
+    return [os.path.join(HERE, f) for f in names]
+
+
+def linked_sources():
+    """Names of the sources in the library as it lies, None when there is no library.  A library without
+    a record of its objects counts as complete."""
+    if not os.path.exists(LIB_PATH):
+        return None
+    manifest = LIB_PATH + ".objects"
+    if not os.path.exists(manifest):
+        return {os.path.basename(s) for s in sources()}
+    with open(manifest, encoding="utf-8") as f:
+        return {os.path.basename(line)[:-2] + ".cu" for line in f.read().splitlines() if line}
 
 
 def _headers_mtime() -> float:
@@ -62,11 +81,14 @@ def _compile(src: str, force: bool, verbose: bool) -> tuple[str, str]:
     return obj, proc.stderr
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    """Compiles what is stale and links; returns the library path."""
+def build(force: bool = False, verbose: bool = False, only=None) -> str:
+    """Compiles what is stale and links; returns the library path.  ``only``: names of the sources a
+    caller needs (they must link among themselves); what is compiled already stays in the library."""
     os.makedirs(OBJ_DIR, exist_ok=True)
     os.makedirs(LIB_DIR, exist_ok=True)
-    srcs = sources()
+    if only is not None:
+        only = set(only) | ((linked_sources() or set()) & {os.path.basename(s) for s in sources()})
+    srcs = sources(only)
     with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, len(srcs) or 1)) as pool:
         results = list(pool.map(lambda s: _compile(s, force, verbose), srcs))
     objs = [o for o, _ in results]

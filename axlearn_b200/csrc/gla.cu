@@ -1,4 +1,4 @@
-// Gated linear attention: a matrix-valued recurrent state with one decay per key channel.
+// Gated linear attention: a matrix-valued recurrent state, every key channel with its own decay.
 //
 // Per head, with q scaled by q_scale, key channel c and value column d:
 //   z_t   = W_a2 (a1 of the projection) + bias              (low-rank gate, [heads * dim])

@@ -4,8 +4,8 @@
   linear distance bias) and a gated linear attention, each RMS-normed (``common/sequence_mixer.py``).
 * Several residual streams with learned read / write / mix weights instead of one residual, branches
   scaled by a constant (``common/hyper_connection.py``).
-* Norm weights stored around zero, SwiGLU feed-forward (optional per layer), a run of layers that may be
-  repeated with the same weights, tied embeddings.
+* Norm weights kept as offsets from one, SwiGLU feed-forward (a layer may lack it), a run of layers that may
+  be repeated with the same weights, tied embeddings.
 
 ``model_config`` takes the dictionary of a checkpoint's ``config.json``; ``parameters`` maps its tensors to
 the model's tree.  Sizes may differ from layer to layer.
@@ -38,6 +38,9 @@ from axlearn_b200.experiments.text.gpt.common import (
 
 ARCHITECTURE = "Sagisun"
 Tensor = torch.Tensor
+# Kernels of an inference process (a first run without a built library compiles these).
+KERNEL_SOURCES = ("flash_fwd.cu", "flash_fwd_v3.cu", "gated_act.cu", "gemm.cu", "gemm_2cta.cu", "gla.cu", "hyper.cu",
+                  "window_attn.cu")
 # A window that never closes (a left mixer without a mask).
 _NO_WINDOW = 1 << 30
 

@@ -17,7 +17,7 @@ from axlearn_b200.common import causal_lm
 from axlearn_b200.common.safetensors_io import read_safetensors
 
 # architecture -> module with ``checkpoint_model_config(config, tensors)`` and
-# ``parameters(model, tensors, dtype=, device=)``.
+# ``parameters(model, tensors, dtype=, device=)`` and ``KERNEL_SOURCES``.
 ARCHITECTURES = {
     "Sagisun": "axlearn_b200.experiments.text.gpt.sagisun",
 }
@@ -41,6 +41,10 @@ def load_model(folder: str, *, dtype: torch.dtype = torch.bfloat16, device: Any 
     if name not in ARCHITECTURES:
         raise ValueError(f"unknown architecture {name!r}; known: {sorted(ARCHITECTURES)}")
     module = importlib.import_module(ARCHITECTURES[name])
+    if device is not None and torch.device(device).type == "cuda":
+        from axlearn_b200.ops import cuda_ops
+
+        cuda_ops.require_sources(module.KERNEL_SOURCES)
     tensors = read_safetensors(os.path.join(folder, "model.safetensors"))
     cfg = module.checkpoint_model_config(config, tensors).set(name="model", dtype=dtype)
     model = cfg.instantiate(parent=None)

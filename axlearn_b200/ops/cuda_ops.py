@@ -42,19 +42,31 @@ def reserve_sms_for_comm(n: int) -> None:
 c_void_p, c_int, c_int64, c_float = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float
 
 
+_required_sources: Optional[frozenset] = None
+
+
+def require_sources(names) -> None:
+    """Declares the ``.cu`` files that this process needs (before its first kernel), so that a first
+    use without a built library compiles those and no others.  Without a declaration: all of them."""
+    global _required_sources
+    _required_sources = frozenset(names) | (_required_sources or frozenset())
+
+
 def lib() -> ctypes.CDLL:
     global _lib_handle
     if _lib_handle is not None:
         return _lib_handle
     with _lib_lock:
         if _lib_handle is None:
-            if not os.path.exists(_LIB_PATH):
-                from axlearn_b200.csrc import build as _build
+            from axlearn_b200.csrc import build as _build
 
-                _build.build()
+            have = _build.linked_sources()
+            needed = _required_sources or {os.path.basename(s) for s in _build.sources()}
+            if have is None or not needed <= have:
+                _build.build(only=_required_sources)
             h = ctypes.CDLL(_LIB_PATH)
             for name in dir(_Sigs):
-                if name.startswith("axb_"):
+                if name.startswith("axb_") and hasattr(h, name):
                     fn = getattr(h, name)
                     fn.argtypes = getattr(_Sigs, name)
                     fn.restype = c_int

@@ -1,4 +1,4 @@
-"""Gated linear attention: a recurrent matrix state with a decay per key channel.
+"""Gated linear attention: a recurrent matrix state whose key channels decay each at their own rate.
 
 Per head: ``S_t = diag(alpha_t) S_(t-1) + k_t v_t^T``, ``o_t = S_t^T (q_t * q_scale)`` with
 ``alpha_t = sigmoid(W_a2 a1_t + b)^(1 / tau)``; then ``rms(o) * norm * silu(gate)`` over the value size.

@@ -101,7 +101,7 @@ def _window_oracle(row, spec, cols):
 
 
 WINDOW_SIZES = [  # heads, kv heads, dim, value dim, window
-    (4, 2, 48, 32, 20), (2, 2, 64, 64, 33), (8, 1, 128, 128, 64), (4, 4, 128, 64, 300), (3, 1, 40, 72, 17),
+    (4, 2, 56, 32, 20), (2, 2, 64, 64, 33), (8, 1, 128, 128, 64), (4, 4, 128, 64, 300), (3, 1, 40, 72, 17),
     (6, 3, 20, 12, 9), (2, 1, 96, 128, 1), (4, 1, 160, 144, 50), (5, 5, 7, 5, 11), (4, 2, 64, 128, 128)]
 
 
@@ -225,7 +225,7 @@ def _gla_oracle(row, cols, a2, bias, norm, spec, state=None):
     return o * oracle.silu(row[:, cols.g:cols.g + o.shape[1]].double()), state
 
 
-GLA_SIZES = [(3, 48, 64, 16), (2, 64, 128, 16), (1, 128, 128, 8), (2, 128, 64, 20), (2, 32, 256, 16), (4, 24, 40, 5),
+GLA_SIZES = [(3, 56, 64, 16), (2, 64, 128, 16), (1, 128, 128, 8), (2, 128, 64, 20), (2, 32, 256, 16), (4, 24, 40, 5),
              (2, 7, 9, 3), (1, 128, 200, 48), (1, 200, 64, 16), (5, 40, 24, 40)]
 
 
@@ -261,7 +261,7 @@ def test_gla_prompt_then_single_tokens(dtype, sizes, tau, z_bias):
             _close(state[r], states[r], 1e-4)
 
 
-@pytest.mark.parametrize("sizes", [(2, 64, 64, 16), (2, 128, 128, 16), (2, 48, 256, 16)])
+@pytest.mark.parametrize("sizes", [(2, 64, 64, 16), (2, 128, 128, 16), (2, 40, 256, 16)])
 @pytest.mark.parametrize("tau", [16.0, 0.5])
 def test_gla_segments_and_portions_agree(sizes, tau):
     heads, dim, vdim, rank = sizes
