@@ -47,7 +47,7 @@ class HyperConnection(BaseLayer):
         norm_offset: float = 1.0
 
     class Parts(NamedTuple):
-        read: Tensor
+        read: Optional[Tensor]
         norm_scale: Tensor
         norm_eps: float
         norm_offset: float
@@ -70,13 +70,40 @@ class HyperConnection(BaseLayer):
                           hyper_ops.StreamWrite(p["mix"], p["write"], cfg.multiplier))
 
 
+class ResidualConnection(BaseLayer):
+    """The ordinary residual as a connection: input ``norm(x)``, ``x <- x + multiplier * y`` (one stream, fp32)."""
+
+    @config_class
+    class Config(BaseLayer.Config):
+        input_dim: Required[int] = REQUIRED
+        num_streams: int = 1
+        multiplier: float = 1.0
+        norm_eps: float = 1e-6
+        norm_offset: float = 0.0
+
+    def __init__(self, cfg, *, parent=None):
+        if cfg.num_streams != 1:
+            raise ValueError("an ordinary residual has one stream")
+        super().__init__(cfg, parent=parent)
+
+    def _create_layer_parameter_specs(self):
+        cfg = self._config
+        return {"norm_scale": vector_spec((cfg.input_dim,), 1.0 - cfg.norm_offset)}
+
+    def forward(self) -> HyperConnection.Parts:
+        cfg = self._config
+        return HyperConnection.Parts(None, self.parameters["norm_scale"], cfg.norm_eps, cfg.norm_offset,
+                                     hyper_ops.PLAIN_WRITE._replace(multiplier=cfg.multiplier))
+
+
 class GatedFeedForward(BaseLayer):
-    """``down(silu(gate x) * up x)`` with gate and up packed in one product."""
+    """``down(act(gate x, up x))`` with gate and up packed in one product; ``gate`` names the activation."""
 
     @config_class
     class Config(BaseLayer.Config):
         input_dim: Required[int] = REQUIRED
         hidden_dim: Required[int] = REQUIRED
+        gate: hyper_ops.Gate = hyper_ops.Gate("silu")
 
     def __init__(self, cfg, *, parent=None):
         super().__init__(cfg, parent=parent)
@@ -91,7 +118,8 @@ class GatedFeedForward(BaseLayer):
         return self._up
 
     def forward(self, x: Tensor) -> Tensor:
-        return self.linear2(hyper_ops.gated_act(self.linear1(x), self._config.hidden_dim, self._up))
+        cfg = self._config
+        return self.linear2(hyper_ops.gated_act(self.linear1(x), cfg.hidden_dim, self._up, cfg.gate))
 
 
 class HyperTransformerLayer(BaseTransformerLayer):
@@ -99,7 +127,7 @@ class HyperTransformerLayer(BaseTransformerLayer):
     class Config(BaseTransformerLayer.Config):
         mixer: Required[InstantiableConfig] = REQUIRED
         feed_forward: Optional[InstantiableConfig] = None
-        connection: HyperConnection.Config = HyperConnection.default_config()
+        connection: InstantiableConfig = HyperConnection.default_config()
 
     def __init__(self, cfg, *, parent=None):
         super().__init__(cfg, parent=parent)
@@ -136,11 +164,13 @@ class HyperStackedTransformerLayer(BaseStackedTransformerLayer):
 
     @config_class
     class Config(BaseStackedTransformerLayer.Config):
-        num_streams: Required[int] = REQUIRED
+        num_streams: int = 1
         # (start, stop, times): layers start .. stop - 1 run `times` times in a row.
         loop: Optional[tuple] = None
         output_norm_eps: float = 1e-6
         output_norm_offset: float = 1.0
+        # Constant factor of the normed output (a logit scale ahead of a linear head).
+        output_multiplier: float = 1.0
 
     def __init__(self, cfg, *, parent=None):
         super().__init__(cfg, parent=parent)
@@ -188,7 +218,8 @@ class HyperStackedTransformerLayer(BaseStackedTransformerLayer):
             new_states[f"run{run}"] = state
         _, h = hyper_ops.hyper_step(
             streams, branch, write=write, read=None, norm_scale=self.parameters["output_norm_scale"],
-            eps=cfg.output_norm_eps, norm_offset=cfg.output_norm_offset, keep_streams=False, **step)
+            eps=cfg.output_norm_eps, norm_offset=cfg.output_norm_offset, keep_streams=False,
+            h_multiplier=cfg.output_multiplier, **step)
         return new_states, self.Output(data=h)
 
     def forward(self, data, *, target_segment_ids=None, target_positions=None, return_aux=None, **kwargs):

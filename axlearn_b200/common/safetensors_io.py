@@ -65,3 +65,48 @@ def write_safetensors(path: str, tensors: Mapping[str, torch.Tensor], metadata: 
         f.write(len(text).to_bytes(8, "little") + text)
         for raw in blobs:
             f.write(raw)
+
+
+class TreeLoader:
+    """Fills a model's parameter tree from a checkpoint's tensors.
+
+    ``tree`` starts as zeros: matrices in ``dtype``, parameters declared fp32 in fp32.  Every tensor is taken
+    with its expected shape; ``finish`` refuses tensors that no part of the model took."""
+
+    def __init__(self, model, tensors, *, dtype):
+        self._tensors, self._used = tensors, set()
+
+        def build(node):
+            if isinstance(node, dict):
+                return {name: build(child) for name, child in node.items()}
+            return torch.zeros(tuple(node.shape), dtype=torch.float32 if node.dtype == torch.float32 else dtype)
+
+        self.tree = build(model.create_parameter_specs_recursively())
+
+    def take(self, name: str, shape) -> torch.Tensor:
+        t = self._tensors[name]
+        if tuple(t.shape) != tuple(shape):
+            raise ValueError(f"{name} has shape {tuple(t.shape)}, expected {tuple(shape)}")
+        self._used.add(name)
+        return t
+
+    @staticmethod
+    def put(dst: torch.Tensor, src: torch.Tensor, row: int = 0) -> None:
+        """``src`` into the top left corner of ``dst`` from ``row`` on (stored sizes may be larger)."""
+        dst[row:row + src.shape[0], :src.shape[1]] = src.to(dst.dtype)
+
+    def fill(self, dst: torch.Tensor, name: str, shape, row: int = 0) -> None:
+        self.put(dst, self.take(name, shape), row)
+
+    def copy(self, dst: torch.Tensor, name: str, shape) -> None:
+        dst.copy_(self.take(name, shape))
+
+    def finish(self, device=None) -> dict:
+        unused = set(self._tensors) - self._used
+        if unused:
+            raise ValueError(f"tensors of no part of the model: {sorted(unused)[:5]} ({len(unused)} in all)")
+
+        def place(node):
+            return {k: place(v) if isinstance(v, dict) else v.to(device) for k, v in node.items()}
+
+        return place(self.tree)

@@ -1,5 +1,5 @@
-"""Sequence mixers over packed projections: gated window attention, gated linear attention, and the two
-side by side.
+"""Sequence mixers over packed projections: gated window attention, gated linear attention and the two side
+by side; latent attention; state-space mixing (Mamba-2).
 
 A mixer names the sections it needs of a token's projection (``sections``), and mixes along the sequence
 given a projection that contains them (``mix``).  So several mixers that read the same input share ONE
@@ -23,7 +23,7 @@ from axlearn_b200.common.config import REQUIRED, Required, config_class
 from axlearn_b200.common.kv_cache import RingKVCache
 from axlearn_b200.common.module import nowrap
 from axlearn_b200.common.param_init import FanAxes, constant_initializer
-from axlearn_b200.ops import gla_ops, hyper_ops, window_ops
+from axlearn_b200.ops import gla_ops, hyper_ops, latent_ops, ssd_ops, window_ops
 from axlearn_b200.ops.hyper_ops import padded
 
 Tensor = torch.Tensor
@@ -77,6 +77,11 @@ class BaseSequenceMixer(BaseLayer):
         if not cfg.packed_input:
             self._columns, width = layout_sections(self.sections())
             self._add_child("i_proj", PaddedLinear.default_config().set(input_dim=cfg.input_dim, output_dim=width))
+
+    @nowrap
+    def columns(self) -> dict:
+        """``{section: first column}`` of the own projection."""
+        return self._columns
 
     @nowrap
     def sections(self) -> list:
@@ -198,6 +203,118 @@ class GatedLinearAttention(BaseSequenceMixer):
         out, state = gla_ops.gated_linear_attention(
             proj, p["gate_weight"].to(proj.dtype), p["gate_bias"], p["norm_scale"], self._spec,
             gla_ops.GlaColumns(**columns), start=start, live=live, state=state)
+        return self.o_proj(out), state
+
+
+class LatentAttention(BaseSequenceMixer):
+    """Attention whose keys and values come from one cached low-rank vector per token, with a rotated key
+    part shared by all heads (``ops/latent_ops.py``)."""
+
+    @config_class
+    class Config(BaseSequenceMixer.Config):
+        num_heads: Required[int] = REQUIRED
+        per_head_dim: Required[int] = REQUIRED    # unrotated
+        rotated_dim: Required[int] = REQUIRED
+        value_dim: Required[int] = REQUIRED
+        kv_rank: Required[int] = REQUIRED
+        scale: Required[float] = REQUIRED
+        rope_dims: Optional[int] = None           # None = rotated_dim
+        rope_theta: float = 10000.0
+        norm_eps: float = 1e-6
+
+    def __init__(self, cfg, *, parent=None):
+        rope_dims = cfg.rotated_dim if cfg.rope_dims is None else cfg.rope_dims
+        if rope_dims % 2 or rope_dims > cfg.rotated_dim:
+            raise ValueError(f"cannot rotate {rope_dims} of {cfg.rotated_dim} dimensions in pairs")
+        self._spec = latent_ops.LatentSpec(
+            heads=cfg.num_heads, dim=cfg.per_head_dim, rot_dim=cfg.rotated_dim, vdim=cfg.value_dim, rank=cfg.kv_rank,
+            rot_dims=rope_dims, rot_base=cfg.rope_theta, scale=cfg.scale, eps=cfg.norm_eps)
+        super().__init__(cfg, parent=parent)
+        self._add_child("o_proj", PaddedLinear.default_config().set(
+            input_dim=cfg.num_heads * cfg.value_dim, output_dim=cfg.input_dim))
+
+    def _create_layer_parameter_specs(self):
+        s = self._spec
+        return {
+            "latent_norm_scale": vector_spec((s.rank,), 1.0),
+            # Keys: [rank, heads * dim], as a per-head matrix its rows are contiguous in both forms of the sum.
+            "key_weight": ParameterSpec(shape=(padded(s.rank, 8), padded(s.heads * s.dim, 32)), mesh_axes=(None, None),
+                                        fan_axes=FanAxes(in_axis=-2, out_axis=-1)),
+            "value_weight": ParameterSpec(shape=(padded(s.heads * s.vdim, 32), padded(s.rank, 8)),
+                                          mesh_axes=(None, None), fan_axes=FanAxes(in_axis=-1, out_axis=-2)),
+        }
+
+    @nowrap
+    def sections(self) -> list:
+        s = self._spec
+        return [("q", s.heads * (s.dim + s.rot_dim)), ("c", s.rank), ("r", s.rot_dim)]
+
+    @nowrap
+    def init_states(self, *, batch_size, max_len, dtype, device=None):
+        return {"latent": torch.zeros((batch_size, max_len, self._spec.row_width), dtype=dtype, device=device)}
+
+    def mix(self, proj, columns, *, start=None, live=None, state=None):
+        p = self.parameters
+        out, state = latent_ops.latent_attention(
+            proj, p["latent_norm_scale"], p["key_weight"], p["value_weight"], self._spec,
+            latent_ops.LatentColumns(**columns), start=start, live=live, cache=state)
+        return self.o_proj(out), state
+
+
+class StateSpaceMixer(BaseSequenceMixer):
+    """Mamba-2: a short convolution, a matrix state with a scalar decay per head, a gated group norm
+    (``ops/ssd_ops.py``)."""
+
+    @config_class
+    class Config(BaseSequenceMixer.Config):
+        num_heads: Required[int] = REQUIRED
+        value_dim: Required[int] = REQUIRED
+        state_dim: Required[int] = REQUIRED
+        num_groups: int = 1
+        conv_taps: int = 4
+        num_norm_groups: int = 1
+        norm_eps: float = 1e-6
+
+    def __init__(self, cfg, *, parent=None):
+        if cfg.num_heads % cfg.num_groups or (cfg.num_heads * cfg.value_dim) % cfg.num_norm_groups:
+            raise ValueError("heads must split into groups, and channels into norm groups, evenly")
+        self._spec = ssd_ops.SsdSpec(
+            heads=cfg.num_heads, vdim=cfg.value_dim, state=cfg.state_dim, groups=cfg.num_groups, taps=cfg.conv_taps,
+            norm_groups=cfg.num_norm_groups, eps=cfg.norm_eps)
+        super().__init__(cfg, parent=parent)
+        self._add_child("o_proj", PaddedLinear.default_config().set(
+            input_dim=self._spec.inner, output_dim=cfg.input_dim))
+
+    def _create_layer_parameter_specs(self):
+        s = self._spec
+        return {
+            "conv_weight": ParameterSpec(shape=(s.taps, s.channels), dtype=torch.float32, mesh_axes=(None, None),
+                                         fan_axes=FanAxes(in_axis=-2, out_axis=-1)),
+            "conv_bias": vector_spec((s.channels,), 0.0),
+            # Steps around 0.05 and decays around exp(-0.05) to begin with.
+            "dt_bias": vector_spec((s.heads,), -3.0),
+            "a_log": vector_spec((s.heads,), 0.0),
+            "d": vector_spec((s.heads,), 1.0),
+            "norm_scale": vector_spec((s.inner,), 1.0),
+        }
+
+    @nowrap
+    def sections(self) -> list:
+        s = self._spec
+        return [("z", s.inner), ("xbc", s.channels), ("dt", s.heads)]
+
+    @nowrap
+    def init_states(self, *, batch_size, max_len, dtype, device=None):
+        s = self._spec
+        return {"ssm": torch.zeros((batch_size, s.heads, s.state, s.vdim), dtype=torch.float32, device=device),
+                "conv": torch.zeros((batch_size, s.taps, s.channels), dtype=dtype, device=device)}
+
+    def mix(self, proj, columns, *, start=None, live=None, state=None):
+        p = self.parameters
+        weights = ssd_ops.SsdWeights(conv_w=p["conv_weight"], conv_b=p["conv_bias"], dt_bias=p["dt_bias"],
+                                     a_log=p["a_log"], d=p["d"], norm_w=p["norm_scale"])
+        out, state = ssd_ops.ssd_mix(proj, weights, self._spec, ssd_ops.SsdColumns(**columns), start=start, live=live,
+                                     state=state)
         return self.o_proj(out), state
 
 

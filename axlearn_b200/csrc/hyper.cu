@@ -7,9 +7,10 @@
 //
 //   y     = branch                                         (one output)
 //         = w * (rms(a) * sa + rms(b) * sb)                (two outputs, rms with its own eps)
-//   x_t  <- sum_s mix[s, t] x_s + m * out[t] * y           (skipped without a branch)
+//   x_t  <- sum_s mix[s, t] x_s + m * out[t] * y           (skipped without a branch; mix = null: identity,
+//                                                           out = null: ones)
 //   u     = sum_s read[s] x_s                              (read = null: plain sum)
-//   h     = u / sqrt(mean(u^2) + eps) * (offset + scale)   (scale = null: h = u, fp32)
+//   h     = u / sqrt(mean(u^2) + eps) * (offset + scale) * h_mult   (scale = null: h = u, fp32)
 //
 // All arithmetic is fp32.  `h` rows are h_ld wide and zero beyond the width.
 #include <cuda_bf16.h>
@@ -24,15 +25,15 @@ struct HyperArgs {
   const void* branch_b;
   const float* scale_a;
   const float* scale_b;
-  const float* mix;      // [S, S] from, to
-  const float* out_w;    // [S]
+  const float* mix;      // [S, S] from, to, or null
+  const float* out_w;    // [S] or null
   const float* read;     // [S] or null
   const float* norm_scale;
   float* streams_out;    // [rows, S, D] or null
   void* h;
   int64_t rows, streams_ld, branch_ld, h_ld;
   int width, num_streams, streams_equal, streams_bf16, act_bf16;
-  float multiplier, pair_weight, pair_eps, eps, norm_offset;
+  float multiplier, pair_weight, pair_eps, eps, norm_offset, h_mult;
 };
 
 constexpr int kMaxStreams = 16;
@@ -115,10 +116,11 @@ __global__ void __launch_bounds__(max_threads(S)) hyper_step_kernel(HyperArgs a)
   const int64_t row = blockIdx.x;
   const bool has_branch = a.branch_a != nullptr;
   if (has_branch)
-    for (int i = threadIdx.x; i < n * n; i += blockDim.x) s_mix[i] = a.mix[i];
+    for (int i = threadIdx.x; i < n * n; i += blockDim.x)
+      s_mix[i] = a.mix != nullptr ? a.mix[i] : (i / n == i % n ? 1.f : 0.f);
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     s_read[i] = a.read != nullptr ? a.read[i] : 1.f;
-    s_out[i] = has_branch ? a.out_w[i] * a.multiplier : 0.f;
+    s_out[i] = has_branch ? (a.out_w != nullptr ? a.out_w[i] : 1.f) * a.multiplier : 0.f;
   }
   __syncthreads();
 
@@ -200,7 +202,7 @@ __global__ void __launch_bounds__(max_threads(S)) hyper_step_kernel(HyperArgs a)
     }
   }
   if (a.norm_scale == nullptr) return;
-  const float inv = rsqrtf(block_sum2(sq, 0.f, scratch).x / a.width + a.eps);
+  const float inv = a.h_mult * rsqrtf(block_sum2(sq, 0.f, scratch).x / a.width + a.eps);
   T* ho = static_cast<T*>(a.h) + row * a.h_ld;
   for (int c = threadIdx.x * V; c < a.width; c += blockDim.x * V) {
     Vec<V> u = load_vec<V>(u_row + c);

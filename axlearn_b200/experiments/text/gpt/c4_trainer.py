@@ -15,7 +15,8 @@ def named_trainer_configs() -> dict:
     from axlearn_b200.experiments.text.gpt import envy  # pylint: disable=import-outside-toplevel
 
     configs.update(envy.trainer_configs())
-    from axlearn_b200.experiments.text.gpt import sagisun  # pylint: disable=import-outside-toplevel
+    from axlearn_b200.experiments.text.gpt import sagisun, zukitar  # pylint: disable=import-outside-toplevel
 
     configs.update(sagisun.trainer_configs())
+    configs.update(zukitar.trainer_configs())
     return configs

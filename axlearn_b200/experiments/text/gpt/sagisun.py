@@ -28,6 +28,7 @@ from axlearn_b200.common.hyper_connection import (
     HyperTransformerLayer,
     PaddedEmbedding,
 )
+from axlearn_b200.common.safetensors_io import TreeLoader
 from axlearn_b200.common.sequence_mixer import GatedLinearAttention, GatedWindowAttention, ParallelMixer
 from axlearn_b200.experiments.text.gpt.common import (
     MESH_AXIS_NAMES,
@@ -93,75 +94,45 @@ def checkpoint_model_config(config: Mapping[str, Any], tensors: Mapping[str, Ten
     return model_config(config, gate_rank=ranks)
 
 
-def _fill(dst: Tensor, src: Tensor, row: int = 0) -> None:
-    dst[row:row + src.shape[0], :src.shape[1]] = src.to(dst.dtype)
-
-
 def parameters(model: causal_lm.Model, tensors: Mapping[str, Tensor], *, dtype: torch.dtype, device=None) -> dict:
     """The model's parameter tree from a checkpoint's tensors: projections packed, matrices zero-padded to
     their stored sizes and in ``dtype``, small vectors in fp32."""
-    used = set()
-
-    def build(specs, at=""):
-        tree = {}
-        for name, spec in specs.items():
-            path = f"{at}/{name}" if at else name
-            if isinstance(spec, dict):
-                tree[name] = build(spec, path)
-            else:
-                tree[name] = torch.zeros(tuple(spec.shape), dtype=torch.float32 if spec.dtype == torch.float32 else dtype)
-        return tree
-
-    def take(name: str, shape) -> Tensor:
-        t = tensors[name]
-        if tuple(t.shape) != tuple(shape):
-            raise ValueError(f"{name} has shape {tuple(t.shape)}, expected {tuple(shape)}")
-        used.add(name)
-        return t
-
-    tree = build(model.create_parameter_specs_recursively())
-    decoder = model.decoder
-    cfg = decoder.config
-    d, stack = cfg.dim, decoder.transformer
-    _fill(tree["decoder"]["emb"]["token_emb"]["weight"], take("embed", (cfg.vocab_size, d)))
-    root = tree["decoder"]["transformer"]
-    root["output_norm_scale"].copy_(take("final.norm", (d,)))
+    loader = TreeLoader(model, tensors, dtype=dtype)
+    cfg = model.decoder.config
+    d, stack = cfg.dim, model.decoder.transformer
+    decoder = loader.tree["decoder"]
+    loader.fill(decoder["emb"]["token_emb"]["weight"], "embed", (cfg.vocab_size, d))
+    root = decoder["transformer"]
+    loader.copy(root["output_norm_scale"], "final.norm", (d,))
     n = stack.config.num_streams
     for i in range(stack.config.num_layers):
         node, layer, pre = root[f"layer{i}"], getattr(stack, f"layer{i}"), f"l{i}."
         for q, name in enumerate(layer.sublayers(), start=1):
             c = node[f"{name}_connection"]
-            c["norm_scale"].copy_(take(f"{pre}norm{q}", (d,)))
-            c["read"].copy_(take(f"{pre}hc{q}.in", (n,)))
-            c["write"].copy_(take(f"{pre}hc{q}.out", (n,)))
-            c["mix"].copy_(take(f"{pre}hc{q}.mix", (n, n)))
+            loader.copy(c["norm_scale"], f"{pre}norm{q}", (d,))
+            loader.copy(c["read"], f"{pre}hc{q}.in", (n,))
+            loader.copy(c["write"], f"{pre}hc{q}.out", (n,))
+            loader.copy(c["mix"], f"{pre}hc{q}.mix", (n, n))
         mixer = layer.mixer
         for side in ("left", "right"):
             sub, child, mpre = getattr(mixer, side), node["mixer"][side], f"{pre}mix.{side}."
             for name, rows in sub.sections():
-                _fill(node["mixer"]["i_proj"]["weight"], take(mpre + name, (rows, d)), mixer.columns()[side][name])
+                loader.fill(node["mixer"]["i_proj"]["weight"], mpre + name, (rows, d), mixer.columns()[side][name])
             s = sub.config
-            _fill(child["o_proj"]["weight"], take(mpre + "o", (d, s.num_heads * s.value_dim)))
-            node["mixer"][f"{side}_norm_scale"].copy_(take(mpre + "out", (d,)))
+            loader.fill(child["o_proj"]["weight"], mpre + "o", (d, s.num_heads * s.value_dim))
+            loader.copy(node["mixer"][f"{side}_norm_scale"], mpre + "out", (d,))
         s, child, mpre = mixer.right.config, node["mixer"]["right"], f"{pre}mix.right."
         keys = s.num_heads * s.per_head_dim
-        _fill(child["gate_weight"], take(mpre + "a2", (keys, s.gate_rank)))
-        child["gate_bias"].copy_(take(mpre + "a2.b", (keys,)))
-        child["norm_scale"].copy_(take(mpre + "norm", (s.value_dim,)))
+        loader.fill(child["gate_weight"], mpre + "a2", (keys, s.gate_rank))
+        loader.copy(child["gate_bias"], mpre + "a2.b", (keys,))
+        loader.copy(child["norm_scale"], mpre + "norm", (s.value_dim,))
         if "feed_forward" in layer.sublayers():
             ff, mlp = layer.feed_forward, node["feed_forward"]
             f = ff.config.hidden_dim
-            _fill(mlp["linear1"]["weight"], take(f"{pre}mlp.gate", (f, d)))
-            _fill(mlp["linear1"]["weight"], take(f"{pre}mlp.up", (f, d)), ff.up_offset())
-            _fill(mlp["linear2"]["weight"], take(f"{pre}mlp.down", (d, f)))
-    unused = set(tensors) - used
-    if unused:
-        raise ValueError(f"tensors of no part of the model: {sorted(unused)[:5]} ({len(unused)} in all)")
-
-    def place(node):
-        return {k: place(v) if isinstance(v, dict) else v.to(device) for k, v in node.items()}
-
-    return place(tree)
+            loader.fill(mlp["linear1"]["weight"], f"{pre}mlp.gate", (f, d))
+            loader.fill(mlp["linear1"]["weight"], f"{pre}mlp.up", (f, d), ff.up_offset())
+            loader.fill(mlp["linear2"]["weight"], f"{pre}mlp.down", (d, f))
+    return loader.finish(device)
 
 
 # ------------------------------------------------------------------------------------------

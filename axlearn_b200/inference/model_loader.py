@@ -20,6 +20,7 @@ from axlearn_b200.common.safetensors_io import read_safetensors
 # ``parameters(model, tensors, dtype=, device=)`` and ``KERNEL_SOURCES``.
 ARCHITECTURES = {
     "Sagisun": "axlearn_b200.experiments.text.gpt.sagisun",
+    "Zukitar": "axlearn_b200.experiments.text.gpt.zukitar",
 }
 
 

@@ -39,9 +39,13 @@ class NormedPair(NamedTuple):
 
 
 class StreamWrite(NamedTuple):
-    mix: Tensor          # [S, S], indexed [from, to]
-    out: Tensor          # [S]
+    mix: Optional[Tensor]          # [S, S], indexed [from, to]; None: the identity
+    out: Optional[Tensor]          # [S]; None: ones
     multiplier: float
+
+
+# The write of an ordinary residual.
+PLAIN_WRITE = StreamWrite(None, None, 1.0)
 
 
 def padded(n: int, multiple: int) -> int:
@@ -61,26 +65,29 @@ def combine_branch(branch: Union[Tensor, NormedPair], width: int) -> Tensor:
     return branch[..., :width].float()
 
 
-def reference_hyper_step(streams, branch, write, read, norm_scale, *, eps, norm_offset, dtype, num_streams, width):
+def reference_hyper_step(streams, branch, write, read, norm_scale, *, eps, norm_offset, dtype, num_streams, width,
+                         h_multiplier=1.0):
     x = streams.float()
     if x.dim() == 3:
         x = x[:, :, None, :].expand(-1, -1, num_streams, -1)
     if branch is not None:
         y = combine_branch(branch, width)
-        x = torch.einsum("btsd,se->bted", x, write.mix.float()) + (
-            write.multiplier * write.out.float())[:, None] * y[:, :, None, :]
+        out = write.out.float() if write.out is not None else torch.ones(num_streams, device=y.device)
+        mixed = x if write.mix is None else torch.einsum("btsd,se->bted", x, write.mix.float())
+        x = mixed + (write.multiplier * out)[:, None] * y[:, :, None, :]
         streams = x
     u = x.sum(dim=2) if read is None else torch.einsum("btsd,s->btd", x, read.float())
     if norm_scale is None:
         return streams, u
-    h = (_rms(u, eps) * (norm_offset + norm_scale.float())).to(dtype)
+    h = (_rms(u, eps) * (norm_offset + norm_scale.float()) * h_multiplier).to(dtype)
     return streams, F.pad(h, (0, padded(width, 8) - width))
 
 
 def hyper_step(streams: Tensor, branch: Optional[Union[Tensor, NormedPair]] = None, *,
                write: Optional[StreamWrite] = None, read: Optional[Tensor] = None,
                norm_scale: Optional[Tensor] = None, eps: float = 1e-6, norm_offset: float = 1.0,
-               num_streams: int, dtype: torch.dtype, keep_streams: bool = True) -> tuple[Optional[Tensor], Tensor]:
+               num_streams: int, dtype: torch.dtype, keep_streams: bool = True,
+               h_multiplier: float = 1.0) -> tuple[Optional[Tensor], Tensor]:
     """``(new streams, next input)``.
 
     streams: ``[B, T, D]`` (all streams equal) or fp32 ``[B, T, S, D]``.  branch / write: the previous
@@ -88,7 +95,7 @@ def hyper_step(streams: Tensor, branch: Optional[Union[Tensor, NormedPair]] = No
     for the plain sum of the streams.  norm_scale: the norm's stored weight, applied as
     ``norm_offset + weight``; None returns the fp32 sum itself.  The next input is ``[B, T, D']`` with
     D' = D rounded up to 8, its padding zero (a matrix-product operand).  ``keep_streams=False`` (the
-    last read of a stack) returns no streams."""
+    last read of a stack) returns no streams.  ``h_multiplier`` scales the normed output."""
     width = streams.shape[-1]
     if branch is not None and write is None:
         raise ValueError("a branch needs its write weights")
@@ -100,9 +107,10 @@ def hyper_step(streams: Tensor, branch: Optional[Union[Tensor, NormedPair]] = No
     on_gpu = dispatch._cuda(*tensors) and not grad  # pylint: disable=protected-access
     if on_gpu and dtype in (torch.bfloat16, torch.float32):
         return _cuda_hyper_step(streams, branch, write, read, norm_scale, eps=eps, norm_offset=norm_offset,
-                                dtype=dtype, num_streams=num_streams, width=width, keep_streams=keep_streams)
+                                dtype=dtype, num_streams=num_streams, width=width, keep_streams=keep_streams,
+                                h_multiplier=h_multiplier)
     new, h = reference_hyper_step(streams, branch, write, read, norm_scale, eps=eps, norm_offset=norm_offset,
-                                  dtype=dtype, num_streams=num_streams, width=width)
+                                  dtype=dtype, num_streams=num_streams, width=width, h_multiplier=h_multiplier)
     return (new if keep_streams else None), h
 
 
@@ -115,7 +123,7 @@ class _Args(ctypes.Structure):
         ("rows", ctypes.c_int64), ("streams_ld", ctypes.c_int64), ("branch_ld", ctypes.c_int64),
         ("h_ld", ctypes.c_int64)] + [(n, ctypes.c_int) for n in (
             "width", "num_streams", "streams_equal", "streams_bf16", "act_bf16")] + [(n, ctypes.c_float) for n in (
-                "multiplier", "pair_weight", "pair_eps", "eps", "norm_offset")]
+                "multiplier", "pair_weight", "pair_eps", "eps", "norm_offset", "h_mult")]
 
 
 _signature_set = False
@@ -130,7 +138,8 @@ def _lib():
         h.axb_hyper_step.argtypes = [ctypes.POINTER(_Args), ctypes.c_void_p]
         h.axb_hyper_step.restype = ctypes.c_int
         h.axb_gated_act.argtypes = ([ctypes.c_void_p] * 2 + [ctypes.c_int64, ctypes.c_int, ctypes.c_int]
-                                    + [ctypes.c_int64] * 2 + [ctypes.c_int, ctypes.c_void_p])
+                                    + [ctypes.c_int64] * 2 + [ctypes.c_int] * 2 + [ctypes.c_float] * 2
+                                    + [ctypes.c_void_p])
         h.axb_gated_act.restype = ctypes.c_int
         _signature_set = True
     return h
@@ -141,7 +150,7 @@ def _f32(t: Optional[Tensor]) -> Optional[Tensor]:
 
 
 def _cuda_hyper_step(streams, branch, write, read, norm_scale, *, eps, norm_offset, dtype, num_streams, width,
-                     keep_streams):
+                     keep_streams, h_multiplier):
     from axlearn_b200.ops import cuda_ops
 
     if num_streams > MAX_STREAMS:
@@ -192,14 +201,41 @@ def _cuda_hyper_step(streams, branch, write, read, norm_scale, *, eps, norm_offs
     a.rows, a.streams_ld = b * t, (streams.stride(1) if equal else num_streams * width)
     a.width, a.num_streams, a.streams_equal = width, num_streams, int(equal)
     a.streams_bf16, a.act_bf16 = int(streams.dtype == torch.bfloat16), int(dtype == torch.bfloat16)
-    a.eps, a.norm_offset = eps, norm_offset
+    a.eps, a.norm_offset, a.h_mult = eps, norm_offset, h_multiplier
     cuda_ops._check(_lib().axb_hyper_step(ctypes.byref(a), cuda_ops._stream()), "axb_hyper_step")  # pylint: disable=protected-access
     return (new if keep_streams else None), h
 
 
-def gated_act(gu: Tensor, width: int, up_offset: int) -> Tensor:
-    """``silu(gate) * up`` of a packed product: gate in columns ``[0, width)``, up from ``up_offset``; the
-    result is ``width`` rounded up to 8 columns wide, zero-padded."""
+class Gate(NamedTuple):
+    """How a gated feed-forward combines its two halves ``g`` and ``u``:
+
+    * ``silu``: ``silu(g) * u``
+    * ``gelu_tanh``: ``gelu(g) * u`` with the tanh form of gelu
+    * ``clamped``: ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u'`` clamped to ``+-limit``
+    """
+
+    kind: str = "silu"
+    limit: float = 0.0
+    alpha: float = 1.702
+
+
+_GATE_KINDS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
+
+
+def gate_values(g: Tensor, u: Tensor, gate: Gate) -> Tensor:
+    if gate.kind == "silu":
+        return F.silu(g) * u
+    if gate.kind == "gelu_tanh":
+        return F.gelu(g, approximate="tanh") * u
+    if gate.kind == "clamped":
+        g, u = g.clamp(max=gate.limit), u.clamp(-gate.limit, gate.limit)
+        return g * torch.sigmoid(gate.alpha * g) * (u + 1)
+    raise ValueError(f"unknown gate {gate.kind!r}")
+
+
+def gated_act(gu: Tensor, width: int, up_offset: int, gate: Gate = Gate()) -> Tensor:
+    """``gate`` applied to a packed product: gate half in columns ``[0, width)``, up half from ``up_offset``;
+    the result is ``width`` rounded up to 8 columns wide, zero-padded."""
     out_ld = padded(width, 8)
     grad = torch.is_grad_enabled() and gu.requires_grad
     if dispatch._cuda(gu) and not grad and gu.dtype in (torch.bfloat16, torch.float32):  # pylint: disable=protected-access
@@ -209,7 +245,8 @@ def gated_act(gu: Tensor, width: int, up_offset: int) -> Tensor:
         out = torch.empty(gu.shape[:-1] + (out_ld,), dtype=gu.dtype, device=gu.device)
         cuda_ops._check(_lib().axb_gated_act(  # pylint: disable=protected-access
             gu.data_ptr(), out.data_ptr(), gu.numel() // gu.shape[-1], width, up_offset, gu.shape[-1], out_ld,
-            int(gu.dtype == torch.bfloat16), cuda_ops._stream()), "axb_gated_act")  # pylint: disable=protected-access
+            int(gu.dtype == torch.bfloat16), _GATE_KINDS[gate.kind], gate.limit, gate.alpha,
+            cuda_ops._stream()), "axb_gated_act")  # pylint: disable=protected-access
         return out
-    y = F.silu(gu[..., :width].float()) * gu[..., up_offset:up_offset + width].float()
+    y = gate_values(gu[..., :width].float(), gu[..., up_offset:up_offset + width].float(), gate)
     return F.pad(y.to(gu.dtype), (0, out_ld - width))
