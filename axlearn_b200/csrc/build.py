@@ -27,7 +27,8 @@ NVCC_FLAGS = [
 ]
 # Everything but these is built with --use_fast_math: their fp32 instantiations are held to fp32
 # accuracy (recurrent decays, norms and softmax of the 32-bit inference mode).
-PRECISE_SOURCES = frozenset({"gated_act.cu", "gla.cu", "hyper.cu", "window_attn.cu"})
+PRECISE_SOURCES = frozenset({"experts.cu", "gated_act.cu", "gla.cu", "hyper.cu", "latent_attn.cu", "skinny_group.cu",
+                             "ssd.cu", "window_attn.cu"})
 
 
 def _nvcc() -> str:

@@ -12,6 +12,9 @@
 //   * masking beyond "causal": segment ids (packed sequences), a sliding window and a tanh
 //     logit cap are applied inside the kernel, and key tiles that no row of a query tile can
 //     see (left of the window, other segments) are skipped on both sides of the range.
+// Latent attention (kLatent): a query / key row is an unrotated part of its head and a rotated part, of the
+// keys one that all heads share; the parts are loaded by tensor maps of their own into neighbouring 64-column
+// blocks, and the key tile has one stage (wide rows: two do not fit beside the queries).
 //
 // Per CTA (640 threads): warp 0 TMA producer, warp 1 MMA issuer (warps 2-3 idle: they keep the
 // softmax warps aligned to warpgroups), warps 4..11 softmax of tile A, warps 12..19 of tile B.  TMEM (512 columns): S_A/P_A 0..127, S_B/P_B 128..255,
@@ -55,17 +58,20 @@ struct FlashFwd3Params {
   const void* gate;    // first gate column of row 0, or null
   int64_t gate_ld, out_ld;
   int vdim, every, bias;
+  int rot_dim;         // kLatent: size of the rotated part (H is the unrotated size)
   float coef;          // query temperature 1 + coef * ln(floor((pos + 1) / every) + 1)
 };
 
-template <int H>
+// H: value columns; HQ: query / key columns; KS: stages of the key tile.
+template <int H, int HQ = H, int KS = 2>
 struct F3Smem {
   static constexpr int kSub = 16384;
   static constexpr int kTile = (H / 64) * kSub;
-  static constexpr int kQ = 0;                  // two tiles
-  static constexpr int kK = kQ + 2 * kTile;     // two stages
-  static constexpr int kV = kK + 2 * kTile;     // two stages
-  static constexpr int kMax = kV + 2 * kTile;   // float [2 parity][2 tiles][2 halves][128]
+  static constexpr int kQTile = (HQ / 64) * kSub;
+  static constexpr int kQ = 0;                   // two tiles
+  static constexpr int kK = kQ + 2 * kQTile;     // KS stages
+  static constexpr int kV = kK + KS * kQTile;    // two stages
+  static constexpr int kMax = kV + 2 * kTile;    // float [2 parity][2 tiles][2 halves][128]
   static constexpr int kSum = kMax + 4096;      // float [2 tiles][2 halves][128]
   static constexpr int kBar = kSum + 2048;
   static constexpr int kTotal = kBar + 256 + 1024;
@@ -129,11 +135,16 @@ __device__ __forceinline__ void exp2_batch8(const uint32_t* s, uint64_t sc2, uin
 // kGated (with kGeneral): scores are scaled per query row (scale * temperature), a linear distance
 // bias is taken off, and the output is multiplied by sigmoid(gate).  Head sizes up to H: the tensor
 // maps of q, k and v have the real head size as inner extent, so TMA fills the rest with zeros.
-template <int H, bool kGeneral, bool kGated = false>
+// kLatent: causal, query / key rows of HQ columns whose last 64 hold the rotated part (tensor maps tmap_qr /
+// tmap_kr, one key head), strided output without a gate.
+template <int H, bool kGeneral, bool kGated = false, bool kLatent = false>
 __global__ void __launch_bounds__(kF3Threads, 1)
 flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                  const __grid_constant__ CUtensorMap tmap_v, FlashFwd3Params p) {
-  using L = F3Smem<H>;
+                  const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_qr,
+                  const __grid_constant__ CUtensorMap tmap_kr, FlashFwd3Params p) {
+  constexpr int HQ = kLatent ? H + 64 : H, KS = kLatent ? 1 : 2;
+  constexpr bool kStrided = kGated || kLatent;  // output rows of out_ld, heads of vdim columns
+  using L = F3Smem<H, HQ, KS>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
@@ -189,6 +200,10 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     tma_prefetch_desc(&tmap_q);
     tma_prefetch_desc(&tmap_k);
     tma_prefetch_desc(&tmap_v);
+    if (kLatent) {
+      tma_prefetch_desc(&tmap_qr);
+      tma_prefetch_desc(&tmap_kr);
+    }
     mbar_init(q_full, 1);
     for (int i = 0; i < 2; ++i) {
       mbar_init(&k_full[i], 1);
@@ -215,28 +230,35 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (elect_one() && any) {
-      mbar_arrive_expect_tx(q_full, 2 * L::kTile);
+      mbar_arrive_expect_tx(q_full, 2 * L::kQTile);
 #pragma unroll
-      for (int x = 0; x < 2; ++x)
+      for (int x = 0; x < 2; ++x) {
 #pragma unroll
         for (int j = 0; j < H / 64; ++j)
-          tma_load_4d(smem + L::kQ + x * L::kTile + j * L::kSub, &tmap_q, q_full, j * 64, head,
+          tma_load_4d(smem + L::kQ + x * L::kQTile + j * L::kSub, &tmap_q, q_full, j * 64, head,
                       t0 + x * 128, batch);
+        if (kLatent)
+          tma_load_4d(smem + L::kQ + x * L::kQTile + H / 64 * L::kSub, &tmap_qr, q_full, 0, head, t0 + x * 128, batch);
+      }
       for (int it = g_lo; it < g_hi; ++it) {
         const int g = it - g_lo;
         const int st = g & 1;
         // K(g) reuses the stage of K(g - 2), last read by the scores issued in iteration g - 3;
         // V(g) reuses the stage of V(g - 2), last read in iteration g - 2.  Completion number k
         // of it_done[1] belongs to iteration 2k - 1, of it_done[0] to iteration 2k.
-        if (g >= 2) {
-          const int k_need = (g & 1) ? (g - 3) / 2 : (g - 2) / 2;
-          if (!mbar_wait(&it_done[(g + 1) & 1], k_need & 1, p.status, kStatusWaitTimeoutProducer)) break;
+        // With one key stage K(g) reuses the stage of K(g - 1), last read by the scores issued in iteration
+        // g - 2: completion number (g - 1) / 2 of it_done[1] for odd g, g / 2 - 1 of it_done[0] for even g.
+        if (KS == 1 ? g >= 1 : g >= 2) {
+          const int k_need = KS == 1 ? ((g & 1) ? (g - 1) / 2 : g / 2 - 1) : ((g & 1) ? (g - 3) / 2 : (g - 2) / 2);
+          if (!mbar_wait(&it_done[(KS == 1 ? g : g + 1) & 1], k_need & 1, p.status, kStatusWaitTimeoutProducer)) break;
         }
-        mbar_arrive_expect_tx(&k_full[st], L::kTile);
+        mbar_arrive_expect_tx(&k_full[st], L::kQTile);
 #pragma unroll
         for (int j = 0; j < H / 64; ++j)
-          tma_load_4d(smem + L::kK + st * L::kTile + j * L::kSub, &tmap_k, &k_full[st], j * 64, kv_head,
+          tma_load_4d(smem + L::kK + (st % KS) * L::kQTile + j * L::kSub, &tmap_k, &k_full[st], j * 64, kv_head,
                       it * 128, batch);
+        if (kLatent)
+          tma_load_4d(smem + L::kK + (st % KS) * L::kQTile + H / 64 * L::kSub, &tmap_kr, &k_full[st], 0, 0, it * 128, batch);
         if (g >= 2) {
           const int v_need = (g & 1) ? (g - 1) / 2 : (g - 2) / 2;
           if (!mbar_wait(&it_done[g & 1], v_need & 1, p.status, kStatusWaitTimeoutProducer)) break;
@@ -265,10 +287,12 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         return d;
       };
       auto issue_qk = [&](int x, int st) {
-        const uint32_t q_lo = desc_lo(smem_u32(smem + L::kQ + x * L::kTile), 16);
-        const uint32_t k_lo = desc_lo(smem_u32(smem + L::kK + st * L::kTile), 16);
+        const uint32_t q_lo = desc_lo(smem_u32(smem + L::kQ + x * L::kQTile), 16);
+        const uint32_t k_lo = desc_lo(smem_u32(smem + L::kK + (st % KS) * L::kQTile), 16);
 #pragma unroll
-        for (int kk = 0; kk < H / 16; ++kk) {
+        for (int kk = 0; kk < HQ / 16; ++kk) {
+          // Steps that hold nothing but the zeros beyond a part's size are left out.
+          if (kLatent && (kk < H / 16 ? kk * 16 >= p.H : (kk - H / 16) * 16 >= p.rot_dim)) continue;
           const uint32_t off = ((kk >> 2) * L::kSub + (kk & 3) * 32) >> 4;
           tc_mma_f16(tmem_base + x * 128, desc(q_lo + off), desc(k_lo + off), idesc_qk, kk > 0 ? 1u : 0u);
         }
@@ -298,10 +322,20 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const uint32_t ph = (g >> 1) & 1;
         const bool has_next = it + 1 < g_hi;
         if (!mbar_wait(&v_full[st], ph, p.status, kStatusWaitTimeoutMma)) break;
-        if (has_next) {
+        // The next key tile is needed by the scores only; with one stage it is on its way until then.
+        bool k_ready = KS == 2;
+        if (has_next && KS == 2) {
           if (!mbar_wait(&k_full[st ^ 1], ((g + 1) >> 1) & 1, p.status, kStatusWaitTimeoutMma)) break;
         }
         tc_fence_after_sync();
+        auto next_keys = [&]() {
+          if (!k_ready) {
+            ok = mbar_wait(&k_full[st ^ 1], ((g + 1) >> 1) & 1, p.status, kStatusWaitTimeoutMma);
+            tc_fence_after_sync();
+            k_ready = true;
+          }
+          return ok;
+        };
         for (int x = 0; x < 2 && ok; ++x) {
           if (it >= lo[x] && it < hi[x]) {
             if (!mbar_wait(&p_full[x], (it - lo[x]) & 1, p.status, kStatusWaitTimeoutMma)) {
@@ -310,10 +344,13 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
             }
             tc_fence_after_sync();
             issue_pv(x, st, it == lo[x]);
-            if (it + 1 < hi[x]) issue_qk(x, st ^ 1);
-            else tc_commit(&pv_done[x]);
+            if (it + 1 < hi[x]) {
+              if (next_keys()) issue_qk(x, st ^ 1);
+            } else {
+              tc_commit(&pv_done[x]);
+            }
           } else if (it + 1 == lo[x] && it + 1 < hi[x]) {
-            issue_qk(x, st ^ 1);  // first score tile of a query tile that starts later
+            if (next_keys()) issue_qk(x, st ^ 1);  // first score tile of a query tile that starts later
           }
         }
         if (!ok) break;
@@ -514,7 +551,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     ex_sum[(x * 2 + half) * 128 + r_in] = l_sum;
     pair_barrier(bar_id);
     l_sum += ex_sum[(x * 2 + (half ^ 1)) * 128 + r_in];
-    if (!kGated && ok && row < p.T) {
+    if (!kStrided && ok && row < p.T) {
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) +
                             ((static_cast<int64_t>(batch) * p.T + row) * p.N + head) * H + half * (H / 2);
       if (half == 0) {
@@ -525,7 +562,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         for (int c = 0; c < H / 2; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
       }
     }
-    if (kGated && ok && nt > 0) {
+    if (kStrided && ok && nt > 0) {
       const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
       const int64_t tok = static_cast<int64_t>(batch) * p.T + row;
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + tok * p.out_ld + head * p.vdim;
@@ -558,7 +595,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         }
       }
     }
-    if (!kGated && ok && nt > 0) {
+    if (!kStrided && ok && nt > 0) {
       const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) +
                             ((static_cast<int64_t>(batch) * p.T + row) * p.N + head) * H + half * (H / 2);
@@ -654,23 +691,14 @@ static int make_packed_map(CUtensorMap* map, const void* base, int B, int L, int
                          CU_TENSOR_MAP_SWIZZLE_128B);
 }
 
-template <int H, bool kGeneral, bool kGated = false>
-static int launch_flash_fwd3(const void* q, const void* k, const void* v, FlashFwd3Params p, cudaStream_t stream) {
-  CUtensorMap tq, tk, tv;
-  if (kGated) {
-    if (make_packed_map(&tq, q, p.B, p.T, p.N, p.H, p.gate_ld)) return -2;
-    if (make_packed_map(&tk, k, p.B, p.S, p.Nkv, p.H, p.gate_ld)) return -2;
-    if (make_packed_map(&tv, v, p.B, p.S, p.Nkv, p.vdim, p.gate_ld)) return -2;
-  } else {
-    if (make_bthd_map(&tq, q, p.B, p.T, p.N, H, 128)) return -2;
-    if (make_bthd_map(&tk, k, p.B, p.S, p.Nkv, H, 128)) return -2;
-    if (make_bthd_map(&tv, v, p.B, p.S, p.Nkv, H, 128)) return -2;
-  }
-  auto kernel = flash_fwd3_kernel<H, kGeneral, kGated>;
+template <int H, bool kGeneral, bool kGated, bool kLatent>
+static int run_flash_fwd3(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tqr,
+                          const CUtensorMap& tkr, const FlashFwd3Params& p, cudaStream_t stream) {
+  constexpr int kSmem = F3Smem<H, kLatent ? H + 64 : H, kLatent ? 1 : 2>::kTotal;
+  auto kernel = flash_fwd3_kernel<H, kGeneral, kGated, kLatent>;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, F3Smem<H>::kTotal) != cudaSuccess)
-      return -3;
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -3;
     // The in-kernel register redistribution only balances if the launch allocates exactly the
     // assumed count per thread; refuse to launch a build for which it does not.
     cudaFuncAttributes attr;
@@ -683,8 +711,23 @@ static int launch_flash_fwd3(const void* q, const void* k, const void* v, FlashF
     configured = true;
   }
   dim3 grid((p.T + 255) / 256, p.N, p.B);
-  kernel<<<grid, kF3Threads, F3Smem<H>::kTotal, stream>>>(tq, tk, tv, p);
+  kernel<<<grid, kF3Threads, kSmem, stream>>>(tq, tk, tv, tqr, tkr, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <int H, bool kGeneral, bool kGated = false>
+static int launch_flash_fwd3(const void* q, const void* k, const void* v, FlashFwd3Params p, cudaStream_t stream) {
+  CUtensorMap tq, tk, tv;
+  if (kGated) {
+    if (make_packed_map(&tq, q, p.B, p.T, p.N, p.H, p.gate_ld)) return -2;
+    if (make_packed_map(&tk, k, p.B, p.S, p.Nkv, p.H, p.gate_ld)) return -2;
+    if (make_packed_map(&tv, v, p.B, p.S, p.Nkv, p.vdim, p.gate_ld)) return -2;
+  } else {
+    if (make_bthd_map(&tq, q, p.B, p.T, p.N, H, 128)) return -2;
+    if (make_bthd_map(&tk, k, p.B, p.S, p.Nkv, H, 128)) return -2;
+    if (make_bthd_map(&tv, v, p.B, p.S, p.Nkv, H, 128)) return -2;
+  }
+  return run_flash_fwd3<H, kGeneral, kGated, false>(tq, tk, tv, tq, tk, p, stream);
 }
 
 }  // namespace axb
@@ -724,7 +767,7 @@ extern "C" int axb_flash_fwd_v3(const void* q, const void* k, const void* v, voi
   p.q_offset = S - T;
   p.window = window;
   p.status = status;
-  p.gate = nullptr, p.gate_ld = 0, p.out_ld = 0, p.vdim = H, p.every = 1, p.bias = 0, p.coef = 0.f;
+  p.gate = nullptr, p.gate_ld = 0, p.out_ld = 0, p.vdim = H, p.every = 1, p.bias = 0, p.rot_dim = 0, p.coef = 0.f;
   const bool general = q_seg != nullptr || window >= 0 || logit_cap > 0.f;
   if (H == 128) {
     return general ? launch_flash_fwd3<128, true>(q, k, v, p, stream) : launch_flash_fwd3<128, false>(q, k, v, p, stream);
@@ -753,7 +796,52 @@ extern "C" int axb_flash_fwd_gated(const void* q, const void* k, const void* v, 
   p.B = B, p.T = T, p.S = T, p.N = N, p.Nkv = Nkv, p.H = dim;
   p.sc = scale * 1.4426950408889634f, p.cap_in = 0.f, p.cap_out = 0.f;
   p.causal = 1, p.q_offset = 0, p.window = window - 1, p.status = status;
-  p.gate = gate, p.gate_ld = ld, p.out_ld = out_ld, p.vdim = vdim, p.every = every, p.bias = bias, p.coef = coef;
+  p.gate = gate, p.gate_ld = ld, p.out_ld = out_ld, p.vdim = vdim, p.every = every, p.bias = bias, p.rot_dim = 0;
+  p.coef = coef;
   if (dim <= 64 && vdim <= 64) return launch_flash_fwd3<64, true, true>(q, k, v, p, stream);
   return launch_flash_fwd3<128, true, true>(q, k, v, p, stream);
+}
+
+// Causal attention of whole prompts whose query rows are [dim | rot_dim] per head, whose unrotated keys are
+// [B, T, k_ld] (head h at column h * dim), whose rotated key part is shared by the heads (rows kr_ld apart,
+// sequences kr_batch apart) and whose values are [B, T, v_ld]; q points at its first column in [B, T, q_ld], out
+// is [B, T, out_ld] with head h at column h * vdim.  All bf16; dim, vdim <= 128, rot_dim <= 64, sizes and pitches
+// multiples of 8, pointers 16-byte aligned.
+extern "C" int axb_flash_fwd_latent(const void* q, const void* k, const void* kr, const void* v, void* out, int B, int T,
+                                    int N, int dim, int rot_dim, int vdim, int64_t q_ld, int64_t k_ld, int64_t kr_ld,
+                                    int64_t kr_batch, int64_t v_ld, int64_t out_ld, float scale, int* status,
+                                    cudaStream_t stream) {
+  using namespace axb;
+  if (B <= 0 || T <= 0 || N <= 0 || dim < 8 || dim > 128 || rot_dim < 8 || rot_dim > 64 || vdim < 8 || vdim > 128 ||
+      ((dim | rot_dim | vdim) % 8) || ((q_ld | k_ld | kr_ld | kr_batch | v_ld | out_ld) % 8) ||
+      out_ld < static_cast<int64_t>(N) * vdim || kr_batch < static_cast<int64_t>(T) * kr_ld)
+    return -10;
+  const uintptr_t align = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) |
+                          reinterpret_cast<uintptr_t>(kr) | reinterpret_cast<uintptr_t>(v) |
+                          reinterpret_cast<uintptr_t>(out);
+  if (align & 15) return -10;
+  FlashFwd3Params p;
+  p.out = out, p.lse = nullptr;
+  p.q_seg = nullptr, p.k_seg = nullptr, p.ranges = nullptr;
+  p.B = B, p.T = T, p.S = T, p.N = N, p.Nkv = N, p.H = dim;
+  p.sc = scale * 1.4426950408889634f, p.cap_in = 0.f, p.cap_out = 0.f;
+  p.causal = 1, p.q_offset = 0, p.window = -1, p.status = status;
+  p.gate = nullptr, p.gate_ld = 0, p.out_ld = out_ld, p.vdim = vdim, p.every = 1, p.bias = 0, p.coef = 0.f;
+  p.rot_dim = rot_dim;
+  auto map = [&](CUtensorMap* m, const void* base, int heads, int cols, int64_t head_ld, int64_t ld, int64_t batch_ld) {
+    uint64_t dims[4] = {static_cast<uint64_t>(cols), static_cast<uint64_t>(heads), static_cast<uint64_t>(T),
+                        static_cast<uint64_t>(B)};
+    uint64_t strides[3] = {static_cast<uint64_t>(head_ld) * 2, static_cast<uint64_t>(ld) * 2,
+                           static_cast<uint64_t>(batch_ld) * 2};
+    uint32_t box[4] = {64, 1, 128, 1};
+    return make_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
+  };
+  const auto* q16 = static_cast<const __nv_bfloat16*>(q);
+  CUtensorMap tq, tk, tv, tqr, tkr;
+  if (map(&tq, q, N, dim, dim + rot_dim, q_ld, T * q_ld) || map(&tqr, q16 + dim, N, rot_dim, dim + rot_dim, q_ld, T * q_ld) ||
+      map(&tk, k, N, dim, dim, k_ld, T * k_ld) || map(&tkr, kr, 1, rot_dim, kr_ld, kr_ld, kr_batch) ||
+      map(&tv, v, N, vdim, vdim, v_ld, T * v_ld))
+    return -2;
+  if (dim <= 64 && vdim <= 64) return run_flash_fwd3<64, false, false, true>(tq, tk, tv, tqr, tkr, p, stream);
+  return run_flash_fwd3<128, false, false, true>(tq, tk, tv, tqr, tkr, p, stream);
 }

@@ -21,6 +21,8 @@
 #include <math.h>
 #include <stdint.h>
 
+#include "mma_sync.cuh"
+
 namespace axb {
 
 struct GlaArgs {
@@ -270,39 +272,9 @@ namespace {
 
 constexpr int kGcTok = 64, kGcThreads = 256;
 
-__device__ __forceinline__ uint32_t sptr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(sptr(p)));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(sptr(p)));
-}
-__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack2(float x, float y) {
-  __nv_bfloat162 p = __floats2bfloat162_rn(x, y);
-  return reinterpret_cast<uint32_t&>(p);
-}
-__device__ __forceinline__ float2 unpack2(uint32_t u) { return __bfloat1622float2(reinterpret_cast<__nv_bfloat162&>(u)); }
-// hi + lo = (x, y) to about 16 mantissa bits.
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack2(x, y);
-  const float2 h = unpack2(hi);
-  lo = pack2(x - h.x, y - h.y);
-}
-__device__ __forceinline__ void cp16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sptr(dst)), "l"(src) : "memory");
-}
 __device__ __forceinline__ void prefetch_row(const __nv_bfloat16* p, int n) {
   for (int c = 0; c < n; c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + c));
 }
-__device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
 // 64 rows of `n` elements (source pitch ld) into a tile of W columns, zero beyond n and beyond `rows`.  A
 // thread keeps its column and walks the rows.
@@ -329,11 +301,6 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16* tile, int pitch, const 
   }
 }
 
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ float lg2(float x) {
   float y;
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

@@ -1,0 +1,525 @@
+// Latent attention: one cached row [latent | rotated key part] per token serves the keys and values of all
+// heads.
+//
+// Cache rows are [row_w] = latent (rank columns, padded to rot_off) then the rotated part (padded); padding is
+// zero.  With queries folded into the latent space (q_lat = W_uk^T q per head) attention is
+//   score = q_row . cache_row * scale,  out_lat = softmax(score) . latents        over j <= position
+// i.e. multi-query attention with a key size of row_w and a value size of rank.
+//
+// `start[b]` tokens are cached already (null: zero; < 0: row not in this step), `live[b]` of the T new ones are
+// valid (null: T).
+//
+//   latent_prep_kernel    norm of the latent, rotation of the key part, cache row; rotation of the queries
+//                         (in place, or into the rows that latent attention reads).
+//   latent_decode_kernel  bf16: 16 or 32 heads of one query token per CTA on the tensor cores, the cached rows
+//                         streamed once through shared memory; long caches are split over CTAs and the last
+//                         one to finish merges.
+//   latent_attn_kernel    any sizes, fp32 or bf16, one CTA per (token, head).
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <math.h>
+#include <stdint.h>
+
+#include "mma_sync.cuh"
+
+namespace axb {
+
+struct LatentArgs {
+  const void* proj;      // queries are rotated in place without qbuf
+  const float* norm_w;   // [rank]
+  const double* freq;    // [rot_dims / 2]
+  void* cache;           // [B, slots, cache_ld]
+  void* lat;             // [B * T, lat_ld] normed latents of the new tokens, or null
+  void* qbuf;            // [B * T, heads, row_w], or null
+  void* out;             // [B * T, heads, out_ld]
+  float* part;           // [B * T, heads, splits, rot_off + 2]
+  int* tickets;          // zero on entry and on exit
+  const int* start;
+  const int* live;
+  int64_t ld, cache_ld, lat_ld, out_ld;
+  int B, T, heads, dim, rot_dim, rot_dims, rank, rot_off, row_w, slots;
+  int q_off, c_off, r_off, splits, act_bf16;
+  float scale, eps;
+};
+
+namespace {
+
+__device__ __forceinline__ float lf(float x) { return x; }
+__device__ __forceinline__ float lf(__nv_bfloat16 x) { return __bfloat162float(x); }
+constexpr float kLog2E = 1.4426950408889634f;
+
+// Position of token t of sequence b, -1 when it takes no part in the step.
+__device__ __forceinline__ int token_position(const LatentArgs& a, int b, int t) {
+  const int start = a.start != nullptr ? a.start[b] : 0;
+  const int live = a.live != nullptr ? a.live[b] : a.T;
+  return start < 0 || t >= live || start + t >= a.slots ? -1 : start + t;
+}
+
+constexpr int kLpThreads = 128;
+
+}  // namespace
+
+template <typename T>
+__global__ void __launch_bounds__(kLpThreads) latent_prep_kernel(LatentArgs a) {
+  extern __shared__ float2 s_turn[];  // (cos, sin) per pair
+  __shared__ float red[kLpThreads / 32];
+  const int t = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  const int64_t row = static_cast<int64_t>(b) * a.T + t;
+  T* src = static_cast<T*>(const_cast<void*>(a.proj)) + row * a.ld;
+  const int pos = token_position(a, b, t);
+  const int half = a.rot_dims / 2;
+  for (int i = tid; i < half; i += kLpThreads) {
+    // The angle is reduced to one turn in double precision.
+    const double turn = 6.283185307179586476925286766559;
+    double angle = max(pos, 0) * a.freq[i];
+    angle -= turn * rint(angle / turn);
+    float s, c;
+    sincosf(static_cast<float>(angle), &s, &c);
+    s_turn[i] = make_float2(c, s);
+  }
+  float sq = 0.f;
+  for (int c = tid; c < a.rank; c += kLpThreads) {
+    const float x = lf(src[a.c_off + c]);
+    sq += x * x;
+  }
+  for (int off = 16; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
+  if ((tid & 31) == 0) red[tid >> 5] = sq;
+  __syncthreads();
+  float total = 0.f;
+#pragma unroll
+  for (int w = 0; w < kLpThreads / 32; ++w) total += red[w];
+  const float inv = 1.f / sqrtf(total / a.rank + a.eps);
+  T* dst = pos >= 0 ? static_cast<T*>(a.cache) + (static_cast<int64_t>(b) * a.slots + pos) * a.cache_ld : nullptr;
+  T* lat = a.lat != nullptr ? static_cast<T*>(a.lat) + row * a.lat_ld : nullptr;
+  for (int c = tid; c < a.rot_off; c += kLpThreads) {
+    const T y = c < a.rank ? T(lf(src[a.c_off + c]) * inv * a.norm_w[c]) : T(0.f);
+    if (dst != nullptr) dst[c] = y;
+    if (lat != nullptr) lat[c] = y;
+  }
+  // Element i of a rotated part, from its unrotated values.
+  auto rotated = [&](const T* x, int i) {
+    if (i >= a.rot_dims) return lf(x[i]);
+    const float2 cs = s_turn[i >> 1];
+    const float u = lf(x[i & ~1]), v = lf(x[i | 1]);
+    return i & 1 ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
+  };
+  const int pad = a.row_w - a.rot_off;
+  if (dst != nullptr)
+    for (int i = tid; i < pad; i += kLpThreads) dst[a.rot_off + i] = i < a.rot_dim ? T(rotated(src + a.r_off, i)) : T(0.f);
+  const int head_w = a.dim + a.rot_dim;
+  if (a.qbuf != nullptr) {
+    T* q = static_cast<T*>(a.qbuf) + row * a.heads * a.row_w + a.rot_off;
+    for (int i = tid; i < a.heads * pad; i += kLpThreads) {
+      const int h = i / pad, c = i % pad;
+      q[static_cast<int64_t>(h) * a.row_w + c] =
+          c < a.rot_dim ? T(rotated(src + a.q_off + h * head_w + a.dim, c)) : T(0.f);
+    }
+  } else {
+    for (int i = tid; i < a.heads * half; i += kLpThreads) {
+      T* x = src + a.q_off + (i / half) * head_w + a.dim + (i % half) * 2;
+      const float2 cs = s_turn[i % half];
+      const float u = lf(x[0]), v = lf(x[1]);
+      x[0] = T(u * cs.x - v * cs.y);
+      x[1] = T(v * cs.x + u * cs.y);
+    }
+  }
+}
+
+constexpr int kLaThreads = 256, kLaKeys = 64, kLaCols = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kLaThreads) latent_attn_kernel(LatentArgs a) {
+  extern __shared__ float s_q[];  // [row_w], times scale * log2(e)
+  __shared__ float s_p[kLaKeys];
+  const int h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int64_t row = blockIdx.y;
+  const int b = static_cast<int>(row / a.T), t = static_cast<int>(row % a.T);
+  T* out = static_cast<T*>(a.out) + (row * a.heads + h) * a.out_ld;
+  const int pos = token_position(a, b, t);
+  if (pos < 0) {
+    for (int c = tid; c < a.rot_off; c += kLaThreads) out[c] = T(0.f);
+    return;
+  }
+  const T* q = static_cast<const T*>(a.qbuf) + (row * a.heads + h) * a.row_w;
+  for (int c = tid; c < a.row_w; c += kLaThreads) s_q[c] = lf(q[c]) * a.scale * kLog2E;
+  const T* keys = static_cast<const T*>(a.cache) + static_cast<int64_t>(b) * a.slots * a.cache_ld;
+  float acc[kLaCols], m = -INFINITY, l = 0.f;
+#pragma unroll
+  for (int i = 0; i < kLaCols; ++i) acc[i] = 0.f;
+  for (int j0 = 0; j0 <= pos; j0 += kLaKeys) {
+    const int n = min(kLaKeys, pos + 1 - j0);
+    __syncthreads();
+    for (int j = warp; j < kLaKeys; j += kLaThreads / 32) {
+      float s = 0.f;
+      if (j < n) {
+        const T* k = keys + static_cast<int64_t>(j0 + j) * a.cache_ld;
+        for (int c = lane; c < a.row_w; c += 32) s += s_q[c] * lf(k[c]);
+      }
+      for (int off = 16; off > 0; off >>= 1) s += __shfl_xor_sync(0xffffffffu, s, off);
+      if (lane == 0) s_p[j] = j < n ? s : -INFINITY;
+    }
+    __syncthreads();
+    float mx = m;
+    for (int j = 0; j < n; ++j) mx = fmaxf(mx, s_p[j]);
+    const float corr = exp2f(m - mx);  // 0 for the first block
+    l *= corr;
+#pragma unroll
+    for (int i = 0; i < kLaCols; ++i) acc[i] *= corr;
+    m = mx;
+    for (int j = 0; j < n; ++j) {
+      const float p = exp2f(s_p[j] - mx);
+      l += p;
+      const T* v = keys + static_cast<int64_t>(j0 + j) * a.cache_ld;
+#pragma unroll
+      for (int i = 0; i < kLaCols; ++i) {
+        const int c = tid + i * kLaThreads;
+        if (c < a.rot_off) acc[i] += p * lf(v[c]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kLaCols; ++i) {
+    const int c = tid + i * kLaThreads;
+    if (c < a.rot_off) out[c] = T(acc[i] / l);
+  }
+}
+
+// ------------------------------------------------------------------------------------------
+// Tensor-core form for a decoding step.
+// ------------------------------------------------------------------------------------------
+namespace {
+
+constexpr int kLdThreads = 256, kLdWarps = 8, kLdKeys = 64, kLdMaxPairs = 4, kLdMaxSplits = 64;
+
+__host__ __device__ constexpr int ld_width(int row_w) { return (row_w + 31) / 32 * 32; }
+
+struct LdSmem {
+  int q, k, stage, s, p, m, l, alpha, flag, total;
+};
+__host__ __device__ inline LdSmem ld_smem(int row_w, int heads) {
+  LdSmem x;
+  const int pitch = (ld_width(row_w) + 8) * 2;
+  x.q = 0;
+  x.k = x.q + heads * pitch;
+  x.stage = kLdKeys * pitch;
+  x.s = x.k + 2 * x.stage;                     // float [heads][68]
+  x.p = x.s + heads * (kLdKeys + 4) * 4;       // bf16 [heads][72]
+  x.m = x.p + heads * (kLdKeys + 8) * 2;
+  x.l = x.m + heads * 4;
+  x.alpha = x.l + heads * 4;
+  x.flag = x.alpha + heads * 4;
+  x.total = x.flag + 16;
+  return x;
+}
+
+}  // namespace
+
+// MT tiles of 16 heads per CTA.
+template <int MT>
+__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(LatentArgs a) {
+  using bf16 = __nv_bfloat16;
+  constexpr int HB = MT * 16;
+  extern __shared__ __align__(16) uint8_t ld_mem[];
+  const LdSmem L = ld_smem(a.row_w, HB);
+  const int WP = ld_width(a.row_w), pitch = WP + 8;
+  bf16* sQ = reinterpret_cast<bf16*>(ld_mem + L.q);
+  float* sS = reinterpret_cast<float*>(ld_mem + L.s);
+  bf16* sP = reinterpret_cast<bf16*>(ld_mem + L.p);
+  float* s_m = reinterpret_cast<float*>(ld_mem + L.m);
+  float* s_l = reinterpret_cast<float*>(ld_mem + L.l);
+  float* s_alpha = reinterpret_cast<float*>(ld_mem + L.alpha);
+  int* s_flag = reinterpret_cast<int*>(ld_mem + L.flag);
+  constexpr int kSP = kLdKeys + 4, kPP = kLdKeys + 8;
+  const int split = blockIdx.x, h0 = blockIdx.y * HB;
+  const int64_t row = blockIdx.z;
+  const int b = static_cast<int>(row / a.T), t = static_cast<int>(row % a.T);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = (lane & 3) * 2;
+  const int nh = min(HB, a.heads - h0);
+  bf16* out = static_cast<bf16*>(a.out) + (row * a.heads + h0) * a.out_ld;
+  const int pos = token_position(a, b, t);
+  if (pos < 0) {
+    if (split == 0)
+      for (int i = tid; i < nh * a.rot_off; i += kLdThreads)
+        out[(i / a.rot_off) * a.out_ld + i % a.rot_off] = __float2bfloat16(0.f);
+    return;
+  }
+  const int count = pos + 1;
+  const int per = ((count + a.splits - 1) / a.splits + kLdKeys - 1) / kLdKeys * kLdKeys;
+  const int j_lo = min(count, split * per), j_hi = min(count, j_lo + per);
+  const bf16* keys = static_cast<const bf16*>(a.cache) + static_cast<int64_t>(b) * a.slots * a.cache_ld;
+  const int chunks = WP / 8, valid = a.row_w / 8;  // 16-byte pieces of a row
+
+  auto load_keys = [&](int j0, int stage) {
+    bf16* dst = reinterpret_cast<bf16*>(ld_mem + L.k + stage * L.stage);
+    for (int i = tid; i < kLdKeys * chunks; i += kLdThreads) {
+      const int r = i / chunks, c = i % chunks;
+      if (c < valid && j0 + r < j_hi)
+        cp16(dst + r * pitch + c * 8, keys + static_cast<int64_t>(j0 + r) * a.cache_ld + c * 8);
+      else
+        *reinterpret_cast<uint4*>(dst + r * pitch + c * 8) = make_uint4(0, 0, 0, 0);
+    }
+  };
+  const bf16* q = static_cast<const bf16*>(a.qbuf) + (row * a.heads + h0) * a.row_w;
+  for (int i = tid; i < HB * chunks; i += kLdThreads) {
+    const int r = i / chunks, c = i % chunks;
+    if (c < valid && r < nh)
+      cp16(sQ + r * pitch + c * 8, q + static_cast<int64_t>(r) * a.row_w + c * 8);
+    else
+      *reinterpret_cast<uint4*>(sQ + r * pitch + c * 8) = make_uint4(0, 0, 0, 0);
+  }
+  load_keys(j_lo, 0);
+  cp_commit();
+  if (tid < HB) s_m[tid] = -INFINITY, s_l[tid] = 0.f;
+
+  const int n_pairs = (a.rank + 15) / 16;  // 16-column tiles of the values, warp, warp + 8, ...
+  float acc[MT][kLdMaxPairs][2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < kLdMaxPairs; ++i)
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[m][i][u][e] = 0.f;
+  const float sc = a.scale * kLog2E;
+
+  for (int j0 = j_lo, it = 0; j0 < j_hi; j0 += kLdKeys, ++it) {
+    const int stage = it & 1;
+    if (j0 + kLdKeys < j_hi) load_keys(j0 + kLdKeys, stage ^ 1);
+    cp_commit();
+    cp_wait_group<1>();
+    __syncthreads();
+    const bf16* sK = reinterpret_cast<const bf16*>(ld_mem + L.k + stage * L.stage);
+    {  // scores of keys [8 warp, + 8)
+      float c0[MT][4], c1[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) c0[m][e] = c1[m][e] = 0.f;
+      const bf16* kp = sK + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 8;
+      const bf16* qp = sQ + (lane & 15) * pitch + (lane >> 4) * 8;
+#pragma unroll 4
+      for (int k = 0; k < WP; k += 32) {
+        uint32_t bk[4];
+        ldsm4(bk, kp + k);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          uint32_t a0[4], a1[4];
+          ldsm4(a0, qp + m * 16 * pitch + k);
+          ldsm4(a1, qp + m * 16 * pitch + k + 16);
+          mma(c0[m], a0, bk[0], bk[1]);
+          mma(c1[m], a1, bk[2], bk[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+          *reinterpret_cast<float2*>(sS + (m * 16 + lr + half * 8) * kSP + warp * 8 + lc) =
+              make_float2((c0[m][half * 2] + c1[m][half * 2]) * sc, (c0[m][half * 2 + 1] + c1[m][half * 2 + 1]) * sc);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {  // 16 lanes per head, 4 keys each
+      const int r = m * 16 + (tid >> 4), c = (tid & 15) * 4;
+      const float4 s4 = *reinterpret_cast<const float4*>(sS + r * kSP + c);
+      float s[4] = {s4.x, s4.y, s4.z, s4.w};
+      float mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (j0 + c + i >= j_hi) s[i] = -INFINITY;
+        mx = fmaxf(mx, s[i]);
+      }
+      for (int off = 8; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      const float old = s_m[r], now = fmaxf(old, mx);  // every block has a visible key: now is finite
+      float p[4], sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        p[i] = exp2f(s[i] - now);
+        sum += p[i];
+      }
+      *reinterpret_cast<uint2*>(sP + r * kPP + c) = make_uint2(pack2(p[0], p[1]), pack2(p[2], p[3]));
+      for (int off = 8; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      __syncwarp();
+      if ((tid & 15) == 0) {
+        const float alpha = exp2f(old - now);
+        s_m[r] = now;
+        s_alpha[r] = alpha;
+        s_l[r] = s_l[r] * alpha + sum;
+      }
+    }
+    __syncthreads();
+    uint32_t ap[MT][4][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float al0 = s_alpha[m * 16 + lr], al1 = s_alpha[m * 16 + lr + 8];
+#pragma unroll
+      for (int i = 0; i < kLdMaxPairs; ++i)
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+          acc[m][i][u][0] *= al0, acc[m][i][u][1] *= al0, acc[m][i][u][2] *= al1, acc[m][i][u][3] *= al1;
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) ldsm4(ap[m][kk], sP + (m * 16 + (lane & 15)) * kPP + kk * 16 + (lane >> 4) * 8);
+    }
+#pragma unroll
+    for (int i = 0; i < kLdMaxPairs; ++i) {
+      const int pair = warp + i * kLdWarps;
+      if (pair < n_pairs) {
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+          uint32_t bv[4];
+          ldsm4t(bv, sK + (kk * 16 + (lane & 15)) * pitch + pair * 16 + (lane >> 4) * 8);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma(acc[m][i][0], ap[m][kk], bv[0], bv[1]);
+            mma(acc[m][i][1], ap[m][kk], bv[2], bv[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();  // the stage may be overwritten
+  }
+  cp_wait_all();
+  __syncthreads();
+
+  const int pw = a.rot_off + 2;
+  float* part = a.splits > 1 ? a.part + ((row * a.heads + h0) * a.splits + split) * pw : nullptr;
+  const int64_t part_head = static_cast<int64_t>(a.splits) * pw;
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < kLdMaxPairs; ++i) {
+      const int pair = warp + i * kLdWarps;
+      if (pair >= n_pairs) continue;
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int r = m * 16 + lr + half * 8, c = pair * 16 + u * 8 + lc;
+          if (r < nh && c < a.rot_off) {  // rot_off is a multiple of 8
+            const float x = acc[m][i][u][half * 2], y = acc[m][i][u][half * 2 + 1];
+            if (part != nullptr) {
+              __stcg(part + r * part_head + c, x);
+              __stcg(part + r * part_head + c + 1, y);
+            } else {
+              const float inv = 1.f / s_l[r];
+              *reinterpret_cast<uint32_t*>(out + r * a.out_ld + c) = pack2(x * inv, y * inv);
+            }
+          }
+        }
+    }
+  if (part == nullptr) return;
+  if (tid < nh) {
+    __stcg(part + tid * part_head + a.rot_off, s_m[tid]);
+    __stcg(part + tid * part_head + a.rot_off + 1, s_l[tid]);
+  }
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {
+    int* ticket = a.tickets + row * gridDim.y + blockIdx.y;
+    const int prev = atomicAdd(ticket, 1);
+    *s_flag = prev == a.splits - 1;
+    if (prev == a.splits - 1) *ticket = 0;
+  }
+  __syncthreads();
+  if (*s_flag == 0) return;
+  __threadfence();
+  // The last CTA merges: weight of every split per head, then the columns.
+  float* s_w = sS;  // [heads][splits]
+  const float* base = a.part + (row * a.heads + h0) * part_head;
+  for (int r = warp; r < nh; r += kLdWarps) {
+    float mx = -INFINITY;
+    for (int s = lane; s < a.splits; s += 32) mx = fmaxf(mx, __ldcg(base + r * part_head + s * pw + a.rot_off));
+    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    float l = 0.f;
+    for (int s = lane; s < a.splits; s += 32) {
+      const float w = exp2f(__ldcg(base + r * part_head + s * pw + a.rot_off) - mx);  // an empty split weighs 0
+      l += w * __ldcg(base + r * part_head + s * pw + a.rot_off + 1);
+      s_w[r * kSP + s] = w;
+    }
+    for (int off = 16; off > 0; off >>= 1) l += __shfl_xor_sync(0xffffffffu, l, off);
+    __syncwarp();
+    for (int s = lane; s < a.splits; s += 32) s_w[r * kSP + s] /= l;
+  }
+  __syncthreads();
+  for (int i = tid; i < nh * a.rot_off; i += kLdThreads) {
+    const int r = i / a.rot_off, c = i % a.rot_off;
+    const float* p = base + r * part_head + c;
+    float x = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < a.splits; ++s) x += s_w[r * kSP + s] * __ldcg(p + static_cast<int64_t>(s) * pw);
+    out[r * a.out_ld + c] = __float2bfloat16(x);
+  }
+}
+
+namespace {
+
+int latent_launched() { return cudaGetLastError() == cudaSuccess ? 0 : -4; }
+
+bool latent_bad(const LatentArgs& a) {
+  return a.B <= 0 || a.T <= 0 || a.heads <= 0 || a.dim <= 0 || a.rot_dim <= 0 || a.rank <= 0 || a.slots <= 0 ||
+         a.rot_dims < 0 || a.rot_dims % 2 || a.rot_dims > a.rot_dim || a.rot_off < a.rank || a.rot_off % 8 || a.row_w % 8 ||
+         a.row_w < a.rot_off + a.rot_dim || a.cache_ld < a.row_w || a.B > 65535;
+}
+
+template <int MT>
+int launch_latent_decode(const LatentArgs& a, cudaStream_t stream) {
+  const int smem = ld_smem(a.row_w, MT * 16).total;
+  static int configured = 48 * 1024;
+  if (smem > configured) {
+    if (smem > 227 * 1024 || cudaFuncSetAttribute(latent_decode_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                  smem) != cudaSuccess)
+      return -3;
+    configured = smem;
+  }
+  const dim3 grid(a.splits, (a.heads + MT * 16 - 1) / (MT * 16), a.B * a.T);
+  latent_decode_kernel<MT><<<grid, kLdThreads, smem, stream>>>(a);
+  return latent_launched();
+}
+
+}  // namespace
+}  // namespace axb
+
+extern "C" int axb_latent_prep(const axb::LatentArgs* args, cudaStream_t stream) {
+  const axb::LatentArgs& a = *args;
+  if (axb::latent_bad(a)) return -10;
+  const size_t smem = sizeof(float2) * (a.rot_dims / 2);
+  if (smem > 48 * 1024) return -10;
+  const dim3 grid(a.T, a.B);
+  if (a.act_bf16)
+    axb::latent_prep_kernel<__nv_bfloat16><<<grid, axb::kLpThreads, smem, stream>>>(a);
+  else
+    axb::latent_prep_kernel<float><<<grid, axb::kLpThreads, smem, stream>>>(a);
+  return axb::latent_launched();
+}
+
+// rank <= 2048.
+extern "C" int axb_latent_attn(const axb::LatentArgs* args, cudaStream_t stream) {
+  const axb::LatentArgs& a = *args;
+  const size_t smem = sizeof(float) * a.row_w;
+  if (axb::latent_bad(a) || a.qbuf == nullptr || a.rot_off > axb::kLaThreads * axb::kLaCols || smem > 40 * 1024 ||
+      static_cast<int64_t>(a.B) * a.T > 65535)
+    return -10;
+  const dim3 grid(a.heads, a.B * a.T);
+  if (a.act_bf16)
+    axb::latent_attn_kernel<__nv_bfloat16><<<grid, axb::kLaThreads, smem, stream>>>(a);
+  else
+    axb::latent_attn_kernel<float><<<grid, axb::kLaThreads, smem, stream>>>(a);
+  return axb::latent_launched();
+}
+
+// Whether the tensor-core kernel takes these sizes.
+extern "C" int axb_latent_decode_supported(int row_w, int rank) {
+  return rank <= 16 * axb::kLdWarps * axb::kLdMaxPairs && axb::ld_smem(row_w, 32).total <= 227 * 1024;
+}
+
+// bf16; splits > 1 needs part and tickets (one per query row and CTA of heads).
+extern "C" int axb_latent_decode(const axb::LatentArgs* args, cudaStream_t stream) {
+  const axb::LatentArgs& a = *args;
+  if (axb::latent_bad(a) || !a.act_bf16 || a.qbuf == nullptr || !axb_latent_decode_supported(a.row_w, a.rank) ||
+      a.splits < 1 || a.splits > axb::kLdMaxSplits || a.cache_ld % 8 || a.out_ld % 8 || a.out_ld < a.rot_off ||
+      static_cast<int64_t>(a.B) * a.T > 65535)
+    return -10;
+  if (a.splits > 1 && (a.part == nullptr || a.tickets == nullptr)) return -11;
+  return a.heads > 16 ? axb::launch_latent_decode<2>(a, stream) : axb::launch_latent_decode<1>(a, stream);
+}

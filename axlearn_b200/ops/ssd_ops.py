@@ -164,7 +164,7 @@ class _Args(ctypes.Structure):
     """Mirrors ``axb::SsdArgs``."""
 
     _fields_ = [(n, ctypes.c_void_p) for n in (
-        "proj", "conv_w", "conv_b", "dt_bias", "a_log", "d", "norm_w", "ssm", "ring", "xbc", "dtv", "v", "out",
+        "proj", "conv_w", "conv_b", "dt_bias", "a_log", "d", "norm_w", "ssm", "ring", "xbc", "v", "out",
         "seg_state", "seg_decay", "start", "live")] + [(n, ctypes.c_int64) for n in (
             "ld", "xbc_ld", "out_ld")] + [(n, ctypes.c_int) for n in (
                 "B", "T", "heads", "vdim", "state", "groups", "taps", "norm_groups", "z_off", "xbc_off", "dt_off",
@@ -249,8 +249,7 @@ def _cuda_ssd_mix(proj, w: SsdWeights, spec: SsdSpec, cols: SsdColumns, *, start
         check(lib.axb_ssd_norm(ctypes.byref(a), stream), "axb_ssd_norm")
         return out, keep
     xbc = torch.empty((b, t, a.xbc_ld), dtype=proj.dtype, device=proj.device)
-    dtv = torch.empty((b, spec.heads, t), dtype=torch.float32, device=proj.device)
-    a.xbc, a.dtv = xbc.data_ptr(), dtv.data_ptr()
+    a.xbc = xbc.data_ptr()
     check(lib.axb_ssd_conv(ctypes.byref(a), stream), "axb_ssd_conv")
     if kernel is None:
         kernel = "chunk" if proj.dtype == torch.bfloat16 and spec.state <= 128 else "scan"
