@@ -91,17 +91,19 @@ __device__ __forceinline__ void scaled_row(const RouteArgs& a, int token, float 
 
 }  // namespace
 
+constexpr int kRsThreads = 512, kRsWarps = kRsThreads / 32;
+
 template <typename T, int EPL>
-__global__ void __launch_bounds__(kRtThreads) route_small_kernel(RouteArgs a) {
+__global__ void __launch_bounds__(kRsThreads) route_small_kernel(RouteArgs a) {
   __shared__ int s_id[kRtMaxPairs], s_place[kRtMaxPairs], s_base[kRtMaxExperts + 1];
   __shared__ float s_w[kRtMaxPairs];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pairs = a.tokens * a.top;
-  for (int t = warp; t < a.tokens; t += kRtWarps)
+  for (int t = warp; t < a.tokens; t += kRsWarps)
     warp_topk<EPL>(a.logits + t * a.logits_ld, a.experts, a.top, [&](int k, int e, float s) {
       if (lane == 0) s_id[t * a.top + k] = e, s_w[t * a.top + k] = s;
     });
   __syncthreads();
-  for (int e = warp; e < a.experts; e += kRtWarps) {
+  for (int e = warp; e < a.experts; e += kRsWarps) {
     int run = 0;
     for (int p0 = 0; p0 < pairs; p0 += 32) {
       const bool mine = p0 + lane < pairs && s_id[p0 + lane] == e;
@@ -127,25 +129,38 @@ __global__ void __launch_bounds__(kRtThreads) route_small_kernel(RouteArgs a) {
   }
   __syncthreads();
   if (blockIdx.x == 0) {
-    for (int e = tid; e <= a.experts; e += kRtThreads) a.offsets[e] = s_base[e];
-    for (int p = tid; p < pairs; p += kRtThreads) a.row_pair[s_base[s_id[p]] + s_place[p]] = p;
+    for (int e = tid; e <= a.experts; e += kRsThreads) a.offsets[e] = s_base[e];
+    for (int p = tid; p < pairs; p += kRsThreads) a.row_pair[s_base[s_id[p]] + s_place[p]] = p;
   }
-  for (int p = blockIdx.x; p < pairs; p += gridDim.x)
-    scaled_row<T>(a, p / a.top, s_w[p], s_base[s_id[p]] + s_place[p], tid, kRtThreads);
+  for (int p = blockIdx.x * 2 + (tid >> 8); p < pairs; p += gridDim.x * 2)
+    scaled_row<T>(a, p / a.top, s_w[p], s_base[s_id[p]] + s_place[p], tid & 255, 256);
 }
 
+constexpr int kRtTokens = 64;  // tokens per CTA of the three-kernel form
+
+// Places come from a count of the CTA's own pairs in shared memory and one addition per (CTA, expert) to the
+// expert's total.
 template <int EPL>
 __global__ void __launch_bounds__(kRtThreads) route_topk_kernel(RouteArgs a) {
-  const int t = blockIdx.x * kRtWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (t >= a.tokens) return;
-  warp_topk<EPL>(a.logits + t * a.logits_ld, a.experts, a.top, [&](int k, int e, float s) {
-    if (lane == 0) {
-      const int p = t * a.top + k;
-      a.ids[p] = e;
-      a.weight[p] = s;
-      a.place[p] = atomicAdd(a.counts + e, 1);
-    }
-  });
+  extern __shared__ int s_count[];  // [experts]: pairs of this CTA, then their first place
+  const int tid = threadIdx.x, lane = tid & 31, t0 = blockIdx.x * kRtTokens;
+  const int t1 = min(a.tokens, t0 + kRtTokens);
+  for (int e = tid; e < a.experts; e += kRtThreads) s_count[e] = 0;
+  __syncthreads();
+  for (int t = t0 + (tid >> 5); t < t1; t += kRtWarps)
+    warp_topk<EPL>(a.logits + t * a.logits_ld, a.experts, a.top, [&](int k, int e, float s) {
+      if (lane == 0) {
+        const int p = t * a.top + k;
+        a.ids[p] = e;
+        a.weight[p] = s;
+        a.place[p] = atomicAdd(s_count + e, 1);
+      }
+    });
+  __syncthreads();
+  for (int e = tid; e < a.experts; e += kRtThreads)
+    if (s_count[e] > 0) s_count[e] = atomicAdd(a.counts + e, s_count[e]);
+  __syncthreads();
+  for (int p = t0 * a.top + tid; p < t1 * a.top; p += kRtThreads) a.place[p] += s_count[a.ids[p]];
 }
 
 // One CTA.
@@ -180,17 +195,46 @@ __global__ void __launch_bounds__(kRtThreads) route_layout_kernel(RouteArgs a) {
   }
 }
 
+// A token's row is read once and written `top` times.
 template <typename T>
 __global__ void __launch_bounds__(kRtThreads) route_gather_kernel(RouteArgs a) {
-  const int p = blockIdx.x * 2 + (threadIdx.x >> 7);
-  if (p >= a.tokens * a.top) return;
-  const int e = a.ids[p], at = a.place[p];
-  const int row = a.offsets[e] + at;
-  scaled_row<T>(a, p / a.top, a.weight[p], row, threadIdx.x & 127, 128);
-  asm volatile("bar.sync %0, 128;" ::"r"(1 + (threadIdx.x >> 7)) : "memory");  // the pair's threads have read place
-  if ((threadIdx.x & 127) == 0) {
+  extern __shared__ int s_row[];  // [top]
+  const int t = blockIdx.x, tid = threadIdx.x;
+  for (int k = tid; k < a.top; k += kRtThreads) {
+    const int p = t * a.top + k, row = a.offsets[a.ids[p]] + a.place[p];
+    s_row[k] = row;
     a.place[p] = row;
     if (a.block == 1) a.row_pair[row] = p;
+  }
+  __syncthreads();
+  const T* src = static_cast<const T*>(a.h) + t * a.h_ld;
+  T* out = static_cast<T*>(a.rows_out);
+  const float* weight = a.weight + static_cast<int64_t>(t) * a.top;
+  if (sizeof(T) == 2 && !((a.h_ld | a.rows_ld | a.width) & 7)) {
+    for (int c = tid * 8; c < a.rows_ld; c += kRtThreads * 8) {
+      float f[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = 0.f;
+      if (c < a.width) {
+        const uint4 u = *reinterpret_cast<const uint4*>(src + c);
+        const uint32_t in[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 x = unpack2(in[i]);
+          f[2 * i] = x.x, f[2 * i + 1] = x.y;
+        }
+      }
+      for (int k = 0; k < a.top; ++k) {
+        const float w = weight[k];
+        *reinterpret_cast<uint4*>(out + s_row[k] * a.rows_ld + c) =
+            make_uint4(pack2(f[0] * w, f[1] * w), pack2(f[2] * w, f[3] * w), pack2(f[4] * w, f[5] * w), pack2(f[6] * w, f[7] * w));
+      }
+    }
+  } else {
+    for (int c = tid; c < a.rows_ld; c += kRtThreads) {
+      const float x = c < a.width ? rf(src[c]) : 0.f;
+      for (int k = 0; k < a.top; ++k) out[s_row[k] * a.rows_ld + c] = T(x * weight[k]);
+    }
   }
 }
 
@@ -229,24 +273,23 @@ bool route_bad(const RouteArgs& a) {
 
 template <int EPL>
 int launch_small(const RouteArgs& a, cudaStream_t stream) {
-  const int pairs = a.tokens * a.top, grid = pairs < 148 ? pairs : 148;
+  const int want = (a.tokens * a.top + 1) / 2, grid = want < 148 ? want : 148;
   if (a.act_bf16)
-    route_small_kernel<__nv_bfloat16, EPL><<<grid, kRtThreads, 0, stream>>>(a);
+    route_small_kernel<__nv_bfloat16, EPL><<<grid, kRsThreads, 0, stream>>>(a);
   else
-    route_small_kernel<float, EPL><<<grid, kRtThreads, 0, stream>>>(a);
+    route_small_kernel<float, EPL><<<grid, kRsThreads, 0, stream>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 template <int EPL>
 int launch_sort(const RouteArgs& a, cudaStream_t stream) {
   if (cudaMemsetAsync(a.counts, 0, sizeof(int) * a.experts, stream) != cudaSuccess) return -4;
-  route_topk_kernel<EPL><<<(a.tokens + kRtWarps - 1) / kRtWarps, kRtThreads, 0, stream>>>(a);
+  route_topk_kernel<EPL><<<(a.tokens + kRtTokens - 1) / kRtTokens, kRtThreads, sizeof(int) * a.experts, stream>>>(a);
   route_layout_kernel<<<1, kRtThreads, 0, stream>>>(a);
-  const int grid = (a.tokens * a.top + 1) / 2;
   if (a.act_bf16)
-    route_gather_kernel<__nv_bfloat16><<<grid, kRtThreads, 0, stream>>>(a);
+    route_gather_kernel<__nv_bfloat16><<<a.tokens, kRtThreads, sizeof(int) * a.top, stream>>>(a);
   else
-    route_gather_kernel<float><<<grid, kRtThreads, 0, stream>>>(a);
+    route_gather_kernel<float><<<a.tokens, kRtThreads, sizeof(int) * a.top, stream>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

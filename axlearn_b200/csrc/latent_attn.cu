@@ -12,8 +12,8 @@
 //   latent_prep_kernel    norm of the latent, rotation of the key part, cache row; rotation of the queries
 //                         (in place, or into the rows that latent attention reads).
 //   latent_decode_kernel  bf16: 16 or 32 heads of one query token per CTA on the tensor cores, the cached rows
-//                         streamed once through shared memory; long caches are split over CTAs and the last
-//                         one to finish merges.
+//                         streamed once through shared memory; long caches are split over CTAs and
+//                         latent_merge_kernel joins the parts.
 //   latent_attn_kernel    any sizes, fp32 or bf16, one CTA per (token, head).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -32,8 +32,8 @@ struct LatentArgs {
   void* lat;             // [B * T, lat_ld] normed latents of the new tokens, or null
   void* qbuf;            // [B * T, heads, row_w], or null
   void* out;             // [B * T, heads, out_ld]
-  float* part;           // [B * T, heads, splits, rot_off + 2]
-  int* tickets;          // zero on entry and on exit
+  float* part;           // [B * T, heads, splits, rot_off] un-normalised sums
+  float* part_ml;        // [B * T, heads, splits, 2] their score maximum (log2) and weight
   const int* start;
   const int* live;
   int64_t ld, cache_ld, lat_ld, out_ld;
@@ -59,8 +59,9 @@ constexpr int kLpThreads = 128;
 
 }  // namespace
 
+// blockIdx.z = 0: the latent and the key part; z > 0: queries of `heads_per` heads.
 template <typename T>
-__global__ void __launch_bounds__(kLpThreads) latent_prep_kernel(LatentArgs a) {
+__global__ void __launch_bounds__(kLpThreads) latent_prep_kernel(LatentArgs a, int heads_per) {
   extern __shared__ float2 s_turn[];  // (cos, sin) per pair
   __shared__ float red[kLpThreads / 32];
   const int t = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
@@ -72,29 +73,10 @@ __global__ void __launch_bounds__(kLpThreads) latent_prep_kernel(LatentArgs a) {
     // The angle is reduced to one turn in double precision.
     const double turn = 6.283185307179586476925286766559;
     double angle = max(pos, 0) * a.freq[i];
-    angle -= turn * rint(angle / turn);
+    angle -= turn * rint(angle * (1.0 / turn));
     float s, c;
     sincosf(static_cast<float>(angle), &s, &c);
     s_turn[i] = make_float2(c, s);
-  }
-  float sq = 0.f;
-  for (int c = tid; c < a.rank; c += kLpThreads) {
-    const float x = lf(src[a.c_off + c]);
-    sq += x * x;
-  }
-  for (int off = 16; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
-  if ((tid & 31) == 0) red[tid >> 5] = sq;
-  __syncthreads();
-  float total = 0.f;
-#pragma unroll
-  for (int w = 0; w < kLpThreads / 32; ++w) total += red[w];
-  const float inv = 1.f / sqrtf(total / a.rank + a.eps);
-  T* dst = pos >= 0 ? static_cast<T*>(a.cache) + (static_cast<int64_t>(b) * a.slots + pos) * a.cache_ld : nullptr;
-  T* lat = a.lat != nullptr ? static_cast<T*>(a.lat) + row * a.lat_ld : nullptr;
-  for (int c = tid; c < a.rot_off; c += kLpThreads) {
-    const T y = c < a.rank ? T(lf(src[a.c_off + c]) * inv * a.norm_w[c]) : T(0.f);
-    if (dst != nullptr) dst[c] = y;
-    if (lat != nullptr) lat[c] = y;
   }
   // Element i of a rotated part, from its unrotated values.
   auto rotated = [&](const T* x, int i) {
@@ -104,19 +86,45 @@ __global__ void __launch_bounds__(kLpThreads) latent_prep_kernel(LatentArgs a) {
     return i & 1 ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
   };
   const int pad = a.row_w - a.rot_off;
-  if (dst != nullptr)
-    for (int i = tid; i < pad; i += kLpThreads) dst[a.rot_off + i] = i < a.rot_dim ? T(rotated(src + a.r_off, i)) : T(0.f);
+  if (blockIdx.z == 0) {
+    float sq = 0.f;
+    for (int c = tid; c < a.rank; c += kLpThreads) {
+      const float x = lf(src[a.c_off + c]);
+      sq += x * x;
+    }
+    for (int off = 16; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
+    if ((tid & 31) == 0) red[tid >> 5] = sq;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int w = 0; w < kLpThreads / 32; ++w) total += red[w];
+    const float inv = 1.f / sqrtf(total / a.rank + a.eps);
+    T* dst = pos >= 0 ? static_cast<T*>(a.cache) + (static_cast<int64_t>(b) * a.slots + pos) * a.cache_ld : nullptr;
+    T* lat = a.lat != nullptr ? static_cast<T*>(a.lat) + row * a.lat_ld : nullptr;
+    for (int c = tid; c < a.rot_off; c += kLpThreads) {
+      const T y = c < a.rank ? T(lf(src[a.c_off + c]) * inv * a.norm_w[c]) : T(0.f);
+      if (dst != nullptr) dst[c] = y;
+      if (lat != nullptr) lat[c] = y;
+    }
+    if (dst != nullptr)
+      for (int i = tid; i < pad; i += kLpThreads) dst[a.rot_off + i] = i < a.rot_dim ? T(rotated(src + a.r_off, i)) : T(0.f);
+    return;
+  }
+  __syncthreads();
   const int head_w = a.dim + a.rot_dim;
+  const int h0 = (blockIdx.z - 1) * heads_per, heads = min(heads_per, a.heads - h0);
+  src += a.q_off + h0 * head_w + a.dim;
   if (a.qbuf != nullptr) {
-    T* q = static_cast<T*>(a.qbuf) + row * a.heads * a.row_w + a.rot_off;
-    for (int i = tid; i < a.heads * pad; i += kLpThreads) {
+    T* q = static_cast<T*>(a.qbuf) + (row * a.heads + h0) * a.row_w + a.rot_off;
+#pragma unroll 4
+    for (int i = tid; i < heads * pad; i += kLpThreads) {
       const int h = i / pad, c = i % pad;
-      q[static_cast<int64_t>(h) * a.row_w + c] =
-          c < a.rot_dim ? T(rotated(src + a.q_off + h * head_w + a.dim, c)) : T(0.f);
+      q[h * a.row_w + c] = c < a.rot_dim ? T(rotated(src + h * head_w, c)) : T(0.f);
     }
   } else {
-    for (int i = tid; i < a.heads * half; i += kLpThreads) {
-      T* x = src + a.q_off + (i / half) * head_w + a.dim + (i % half) * 2;
+#pragma unroll 4
+    for (int i = tid; i < heads * half; i += kLpThreads) {
+      T* x = src + (i / half) * head_w + (i % half) * 2;
       const float2 cs = s_turn[i % half];
       const float u = lf(x[0]), v = lf(x[1]);
       x[0] = T(u * cs.x - v * cs.y);
@@ -131,8 +139,8 @@ template <typename T>
 __global__ void __launch_bounds__(kLaThreads) latent_attn_kernel(LatentArgs a) {
   extern __shared__ float s_q[];  // [row_w], times scale * log2(e)
   __shared__ float s_p[kLaKeys];
-  const int h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int64_t row = blockIdx.y;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int64_t row = blockIdx.x;
   const int b = static_cast<int>(row / a.T), t = static_cast<int>(row % a.T);
   T* out = static_cast<T*>(a.out) + (row * a.heads + h) * a.out_ld;
   const int pos = token_position(a, b, t);
@@ -194,7 +202,7 @@ constexpr int kLdThreads = 256, kLdWarps = 8, kLdKeys = 64, kLdMaxPairs = 4, kLd
 __host__ __device__ constexpr int ld_width(int row_w) { return (row_w + 31) / 32 * 32; }
 
 struct LdSmem {
-  int q, k, stage, s, p, m, l, alpha, flag, total;
+  int q, k, stage, s, p, m, l, alpha, total;
 };
 __host__ __device__ inline LdSmem ld_smem(int row_w, int heads) {
   LdSmem x;
@@ -207,8 +215,7 @@ __host__ __device__ inline LdSmem ld_smem(int row_w, int heads) {
   x.m = x.p + heads * (kLdKeys + 8) * 2;
   x.l = x.m + heads * 4;
   x.alpha = x.l + heads * 4;
-  x.flag = x.alpha + heads * 4;
-  x.total = x.flag + 16;
+  x.total = x.alpha + heads * 4;
   return x;
 }
 
@@ -228,10 +235,9 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(LatentArgs
   float* s_m = reinterpret_cast<float*>(ld_mem + L.m);
   float* s_l = reinterpret_cast<float*>(ld_mem + L.l);
   float* s_alpha = reinterpret_cast<float*>(ld_mem + L.alpha);
-  int* s_flag = reinterpret_cast<int*>(ld_mem + L.flag);
   constexpr int kSP = kLdKeys + 4, kPP = kLdKeys + 8;
-  const int split = blockIdx.x, h0 = blockIdx.y * HB;
-  const int64_t row = blockIdx.z;
+  const int split = blockIdx.y, h0 = blockIdx.z * HB;
+  const int64_t row = blockIdx.x;
   const int b = static_cast<int>(row / a.T), t = static_cast<int>(row % a.T);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = (lane & 3) * 2;
   const int nh = min(HB, a.heads - h0);
@@ -243,20 +249,28 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(LatentArgs
         out[(i / a.rot_off) * a.out_ld + i % a.rot_off] = __float2bfloat16(0.f);
     return;
   }
-  const int count = pos + 1;
-  const int per = ((count + a.splits - 1) / a.splits + kLdKeys - 1) / kLdKeys * kLdKeys;
-  const int j_lo = min(count, split * per), j_hi = min(count, j_lo + per);
+  // Whole tiles of keys, shared out evenly over the splits.
+  const int count = pos + 1, tiles = (count + kLdKeys - 1) / kLdKeys;
+  const int j_lo = static_cast<int>(static_cast<int64_t>(split) * tiles / a.splits) * kLdKeys;
+  const int j_hi = min(count, static_cast<int>(static_cast<int64_t>(split + 1) * tiles / a.splits) * kLdKeys);
   const bf16* keys = static_cast<const bf16*>(a.cache) + static_cast<int64_t>(b) * a.slots * a.cache_ld;
   const int chunks = WP / 8, valid = a.row_w / 8;  // 16-byte pieces of a row
 
+  // A warp takes every eighth row, its lanes the pieces of the row.
   auto load_keys = [&](int j0, int stage) {
-    bf16* dst = reinterpret_cast<bf16*>(ld_mem + L.k + stage * L.stage);
-    for (int i = tid; i < kLdKeys * chunks; i += kLdThreads) {
-      const int r = i / chunks, c = i % chunks;
-      if (c < valid && j0 + r < j_hi)
-        cp16(dst + r * pitch + c * 8, keys + static_cast<int64_t>(j0 + r) * a.cache_ld + c * 8);
-      else
-        *reinterpret_cast<uint4*>(dst + r * pitch + c * 8) = make_uint4(0, 0, 0, 0);
+    bf16* dst = reinterpret_cast<bf16*>(ld_mem + L.k + stage * L.stage) + warp * pitch;
+    const bf16* src = keys + static_cast<int64_t>(j0 + warp) * a.cache_ld;
+#pragma unroll
+    for (int r = 0; r < kLdKeys / kLdWarps; ++r) {
+      const bool in = j0 + warp + r * kLdWarps < j_hi;
+      for (int c = lane; c < chunks; c += 32) {
+        if (in && c < valid)
+          cp16(dst + c * 8, src + c * 8);
+        else
+          *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0, 0, 0, 0);
+      }
+      dst += kLdWarps * pitch;
+      src += kLdWarps * a.cache_ld;
     }
   };
   const bf16* q = static_cast<const bf16*>(a.qbuf) + (row * a.heads + h0) * a.row_w;
@@ -382,9 +396,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(LatentArgs
   cp_wait_all();
   __syncthreads();
 
-  const int pw = a.rot_off + 2;
-  float* part = a.splits > 1 ? a.part + ((row * a.heads + h0) * a.splits + split) * pw : nullptr;
-  const int64_t part_head = static_cast<int64_t>(a.splits) * pw;
+  const int64_t first = (row * a.heads + h0) * a.splits + split;  // this split of the CTA's first head
+  float* part = a.splits > 1 ? a.part + first * a.rot_off : nullptr;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -399,8 +412,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(LatentArgs
           if (r < nh && c < a.rot_off) {  // rot_off is a multiple of 8
             const float x = acc[m][i][u][half * 2], y = acc[m][i][u][half * 2 + 1];
             if (part != nullptr) {
-              __stcg(part + r * part_head + c, x);
-              __stcg(part + r * part_head + c + 1, y);
+              *reinterpret_cast<float2*>(part + static_cast<int64_t>(r) * a.splits * a.rot_off + c) = make_float2(x, y);
             } else {
               const float inv = 1.f / s_l[r];
               *reinterpret_cast<uint32_t*>(out + r * a.out_ld + c) = pack2(x * inv, y * inv);
@@ -408,47 +420,51 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(LatentArgs
           }
         }
     }
-  if (part == nullptr) return;
-  if (tid < nh) {
-    __stcg(part + tid * part_head + a.rot_off, s_m[tid]);
-    __stcg(part + tid * part_head + a.rot_off + 1, s_l[tid]);
-  }
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {
-    int* ticket = a.tickets + row * gridDim.y + blockIdx.y;
-    const int prev = atomicAdd(ticket, 1);
-    *s_flag = prev == a.splits - 1;
-    if (prev == a.splits - 1) *ticket = 0;
-  }
-  __syncthreads();
-  if (*s_flag == 0) return;
-  __threadfence();
-  // The last CTA merges: weight of every split per head, then the columns.
-  float* s_w = sS;  // [heads][splits]
-  const float* base = a.part + (row * a.heads + h0) * part_head;
-  for (int r = warp; r < nh; r += kLdWarps) {
-    float mx = -INFINITY;
-    for (int s = lane; s < a.splits; s += 32) mx = fmaxf(mx, __ldcg(base + r * part_head + s * pw + a.rot_off));
-    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-    float l = 0.f;
-    for (int s = lane; s < a.splits; s += 32) {
-      const float w = exp2f(__ldcg(base + r * part_head + s * pw + a.rot_off) - mx);  // an empty split weighs 0
-      l += w * __ldcg(base + r * part_head + s * pw + a.rot_off + 1);
-      s_w[r * kSP + s] = w;
+  if (part != nullptr && tid < nh)
+    *reinterpret_cast<float2*>(a.part_ml + (first + static_cast<int64_t>(tid) * a.splits) * 2) = make_float2(s_m[tid], s_l[tid]);
+}
+
+// One CTA per (query row, head): parts weighted by their maxima, four columns per thread.
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a) {
+  __shared__ float s_w[kLdMaxSplits];
+  const int64_t row = blockIdx.x;
+  const int h = blockIdx.y, tid = threadIdx.x;
+  if (token_position(a, static_cast<int>(row / a.T), static_cast<int>(row % a.T)) < 0) return;
+  const int64_t first = (row * a.heads + h) * a.splits;
+  if (tid < 32) {
+    float m[kLdMaxSplits / 32], l[kLdMaxSplits / 32], mx = -INFINITY, total = 0.f;
+#pragma unroll
+    for (int i = 0; i < kLdMaxSplits / 32; ++i) {
+      m[i] = -INFINITY, l[i] = 0.f;
+      if (tid + i * 32 < a.splits) {
+        const float2 ml = *reinterpret_cast<const float2*>(a.part_ml + (first + tid + i * 32) * 2);
+        m[i] = ml.x, l[i] = ml.y;
+      }
+      mx = fmaxf(mx, m[i]);
     }
-    for (int off = 16; off > 0; off >>= 1) l += __shfl_xor_sync(0xffffffffu, l, off);
-    __syncwarp();
-    for (int s = lane; s < a.splits; s += 32) s_w[r * kSP + s] /= l;
+    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+#pragma unroll
+    for (int i = 0; i < kLdMaxSplits / 32; ++i) {
+      m[i] = exp2f(m[i] - mx);  // a split without keys weighs 0
+      total += m[i] * l[i];
+    }
+    for (int off = 16; off > 0; off >>= 1) total += __shfl_xor_sync(0xffffffffu, total, off);
+#pragma unroll
+    for (int i = 0; i < kLdMaxSplits / 32; ++i)
+      if (tid + i * 32 < a.splits) s_w[tid + i * 32] = m[i] / total;
   }
   __syncthreads();
-  for (int i = tid; i < nh * a.rot_off; i += kLdThreads) {
-    const int r = i / a.rot_off, c = i % a.rot_off;
-    const float* p = base + r * part_head + c;
-    float x = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < a.splits; ++s) x += s_w[r * kSP + s] * __ldcg(p + static_cast<int64_t>(s) * pw);
-    out[r * a.out_ld + c] = __float2bfloat16(x);
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (row * a.heads + h) * a.out_ld;
+  for (int c = tid * 4; c < a.rot_off; c += 128 * 4) {
+    const float* p = a.part + first * a.rot_off + c;
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < a.splits; ++s) {
+      const float4 v = *reinterpret_cast<const float4*>(p + static_cast<int64_t>(s) * a.rot_off);
+      const float w = s_w[s];
+      x.x += w * v.x, x.y += w * v.y, x.z += w * v.z, x.w += w * v.w;
+    }
+    *reinterpret_cast<uint2*>(out + c) = make_uint2(pack2(x.x, x.y), pack2(x.z, x.w));
   }
 }
 
@@ -472,8 +488,9 @@ int launch_latent_decode(const LatentArgs& a, cudaStream_t stream) {
       return -3;
     configured = smem;
   }
-  const dim3 grid(a.splits, (a.heads + MT * 16 - 1) / (MT * 16), a.B * a.T);
+  const dim3 grid(a.B * a.T, a.splits, (a.heads + MT * 16 - 1) / (MT * 16));
   latent_decode_kernel<MT><<<grid, kLdThreads, smem, stream>>>(a);
+  if (a.splits > 1) latent_merge_kernel<<<dim3(a.B * a.T, a.heads), 128, 0, stream>>>(a);
   return latent_launched();
 }
 
@@ -485,11 +502,13 @@ extern "C" int axb_latent_prep(const axb::LatentArgs* args, cudaStream_t stream)
   if (axb::latent_bad(a)) return -10;
   const size_t smem = sizeof(float2) * (a.rot_dims / 2);
   if (smem > 48 * 1024) return -10;
-  const dim3 grid(a.T, a.B);
+  // Few tokens: the heads side by side; many: fewer copies of the trigonometry.
+  const int heads_per = static_cast<int64_t>(a.B) * a.T <= 1024 ? 4 : 32;
+  const dim3 grid(a.T, a.B, 1 + (a.heads + heads_per - 1) / heads_per);
   if (a.act_bf16)
-    axb::latent_prep_kernel<__nv_bfloat16><<<grid, axb::kLpThreads, smem, stream>>>(a);
+    axb::latent_prep_kernel<__nv_bfloat16><<<grid, axb::kLpThreads, smem, stream>>>(a, heads_per);
   else
-    axb::latent_prep_kernel<float><<<grid, axb::kLpThreads, smem, stream>>>(a);
+    axb::latent_prep_kernel<float><<<grid, axb::kLpThreads, smem, stream>>>(a, heads_per);
   return axb::latent_launched();
 }
 
@@ -498,9 +517,9 @@ extern "C" int axb_latent_attn(const axb::LatentArgs* args, cudaStream_t stream)
   const axb::LatentArgs& a = *args;
   const size_t smem = sizeof(float) * a.row_w;
   if (axb::latent_bad(a) || a.qbuf == nullptr || a.rot_off > axb::kLaThreads * axb::kLaCols || smem > 40 * 1024 ||
-      static_cast<int64_t>(a.B) * a.T > 65535)
+      a.heads > 65535 || static_cast<int64_t>(a.B) * a.T > 0x7fffffff)
     return -10;
-  const dim3 grid(a.heads, a.B * a.T);
+  const dim3 grid(a.B * a.T, a.heads);
   if (a.act_bf16)
     axb::latent_attn_kernel<__nv_bfloat16><<<grid, axb::kLaThreads, smem, stream>>>(a);
   else
@@ -513,13 +532,13 @@ extern "C" int axb_latent_decode_supported(int row_w, int rank) {
   return rank <= 16 * axb::kLdWarps * axb::kLdMaxPairs && axb::ld_smem(row_w, 32).total <= 227 * 1024;
 }
 
-// bf16; splits > 1 needs part and tickets (one per query row and CTA of heads).
+// bf16; splits > 1 needs part and part_ml.
 extern "C" int axb_latent_decode(const axb::LatentArgs* args, cudaStream_t stream) {
   const axb::LatentArgs& a = *args;
   if (axb::latent_bad(a) || !a.act_bf16 || a.qbuf == nullptr || !axb_latent_decode_supported(a.row_w, a.rank) ||
       a.splits < 1 || a.splits > axb::kLdMaxSplits || a.cache_ld % 8 || a.out_ld % 8 || a.out_ld < a.rot_off ||
-      static_cast<int64_t>(a.B) * a.T > 65535)
+      a.heads > 65535 || static_cast<int64_t>(a.B) * a.T > 0x7fffffff)
     return -10;
-  if (a.splits > 1 && (a.part == nullptr || a.tickets == nullptr)) return -11;
+  if (a.splits > 1 && (a.part == nullptr || a.part_ml == nullptr)) return -11;
   return a.heads > 16 ? axb::launch_latent_decode<2>(a, stream) : axb::launch_latent_decode<1>(a, stream);
 }

@@ -17,11 +17,13 @@
 //   ssd_scan_kernel      token by token with the state in registers: fp32, and large states.
 //   ssd_decode_kernel    one token per sequence: convolution, state update and read-out; streams the state
 //                        once.  The ring slot that is written is not one that the step reads.
-//   ssd_norm_kernel      the group norm over the gated outputs `v`.
+//   ssd_norm_kernel      gate and group norm of the outputs `y`.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
 #include <stdint.h>
+
+#include <type_traits>
 
 #include "mma_sync.cuh"
 
@@ -38,7 +40,7 @@ struct SsdArgs {
   float* ssm;            // [B, H, N, P]
   void* ring;            // [B, taps, channels]
   void* xbc;             // [B, T, xbc_ld] convolved channels (prompts)
-  void* v;               // [B, T, inner] gated outputs ahead of the norm
+  void* y;               // [B, T, inner] outputs ahead of the gate
   void* out;             // [B, T, out_ld]
   float* seg_state;      // [B, H, segments, N, P] (segmented prompts)
   float* seg_decay;      // [B, H, segments], log2
@@ -54,7 +56,11 @@ namespace {
 
 __device__ __forceinline__ float sf(float x) { return x; }
 __device__ __forceinline__ float sf(__nv_bfloat16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// x * sigmoid(x); of bf16 activations to well below their rounding.
+__device__ __forceinline__ float silu_t(float x, float) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu_t(float x, __nv_bfloat16) {
+  return __fdividef(x, 1.f + ex2(-x * 1.4426950408889634f));
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 __device__ __forceinline__ bool ssd_inactive(const SsdArgs& a, int b) {
@@ -146,7 +152,7 @@ __global__ void __launch_bounds__(kConvThreads) ssd_conv_kernel(SsdArgs a) {
         for (int i = 0; i < V; ++i) acc[i] += a.conv_w[static_cast<int64_t>(j) * channels + c + i] * x[i];
       }
 #pragma unroll
-      for (int i = 0; i < V; ++i) acc[i] = silu_f(acc[i]);
+      for (int i = 0; i < V; ++i) acc[i] = silu_t(acc[i], T(0.f));
       store_v<V>(dst + t * a.xbc_ld, acc);
     }
     return;
@@ -159,22 +165,47 @@ __global__ void __launch_bounds__(kConvThreads) ssd_conv_kernel(SsdArgs a) {
     for (int i = 0; i < V; ++i) w[j][i] = a.conv_w[static_cast<int64_t>(j) * channels + c + i];
 #pragma unroll
   for (int j = 0; j < K - 1; ++j) input(t0 - K + 1 + j, x[j + 1]);
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-#pragma unroll
-    for (int j = 0; j < K - 1; ++j)
-#pragma unroll
-      for (int i = 0; i < V; ++i) x[j][i] = x[j + 1][i];
-    load_v<V>(src + t * a.ld, x[K - 1]);
+  auto one = [&](int t) {  // x[K - 1] holds the token's input
     float acc[V];
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       acc[i] = bias[i];
 #pragma unroll
       for (int j = 0; j < K; ++j) acc[i] += w[j][i] * x[j][i];
-      acc[i] = silu_f(acc[i]);
+      acc[i] = silu_t(acc[i], T(0.f));
     }
     store_v<V>(dst + t * a.xbc_ld, acc);
+  };
+  auto shift = [&]() {
+#pragma unroll
+    for (int j = 0; j < K - 1; ++j)
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[j][i] = x[j + 1][i];
+  };
+  constexpr int kBatch = 8;  // tokens whose loads are in flight together
+  int t = t0;
+  if (sizeof(T) == 2 && V == 8) {
+    for (; t + kBatch <= t1; t += kBatch) {
+      uint4 raw[kBatch];
+#pragma unroll
+      for (int u = 0; u < kBatch; ++u) raw[u] = *reinterpret_cast<const uint4*>(src + (t + u) * a.ld);
+#pragma unroll
+      for (int u = 0; u < kBatch; ++u) {
+        shift();
+        const uint32_t r[4] = {raw[u].x, raw[u].y, raw[u].z, raw[u].w};
+#pragma unroll
+        for (int i = 0; i < V / 2; ++i) {
+          const float2 f = unpack2(r[i % 4]);
+          x[K - 1][2 * i] = f.x, x[K - 1][2 * i + 1] = f.y;
+        }
+        one(t + u);
+      }
+    }
+  }
+  for (; t < t1; ++t) {
+    shift();
+    load_v<V>(src + t * a.ld, x[K - 1]);
+    one(t);
   }
 }
 
@@ -189,20 +220,48 @@ __global__ void ssd_ring_kernel(SsdArgs a) {
   for (int t = max(0, live - a.taps); t < live; ++t) ring[static_cast<int64_t>((start + t) % a.taps) * channels] = src[t * a.ld];
 }
 
-// rms of v over one norm group, times the weight; columns [inner, out_ld) are written as zeros.
-template <typename T, int V>
+// y silu(z), its rms over one norm group, times the weight; columns [inner, out_ld) are written as zeros.  NV > 0:
+// a thread holds its NV vectors between the two passes; NV = 0: any width, computed twice.
+template <typename T, int V, int NV>
 __global__ void __launch_bounds__(256) ssd_norm_kernel(SsdArgs a) {
   const int inner = a.heads * a.vdim, width = inner / a.norm_groups, c0 = blockIdx.y * width;
   const int64_t row = blockIdx.x;
-  const T* v = static_cast<const T*>(a.v) + row * inner + c0;
+  const T* y = static_cast<const T*>(a.y) + row * inner + c0;
+  const T* z = static_cast<const T*>(a.proj) + row * a.ld + a.z_off + c0;
   T* out = static_cast<T*>(a.out) + row * a.out_ld + c0;
   __shared__ float red[8];
-  float sq = 0.f;
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
-    float f[V];
-    load_v<V>(v + c, f);
+  auto gated = [&](int c, float (&f)[V]) {
+    float g[V];
+    load_v<V>(y + c, f);
+    load_v<V>(z + c, g);
 #pragma unroll
-    for (int i = 0; i < V; ++i) sq += f[i] * f[i];
+    for (int i = 0; i < V; ++i) f[i] *= silu_t(g[i], T(0.f));
+  };
+  auto write = [&](int c, float (&f)[V], float inv) {
+    float w[V];
+    load_v<V>(a.norm_w + c0 + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] *= inv * w[i];
+    store_v<V>(out + c, f);
+  };
+  float sq = 0.f;
+  float keep[NV ? NV : 1][V];
+  if (NV) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = (k * blockDim.x + threadIdx.x) * V;
+      if (c < width) {
+        gated(c, keep[k]);
+#pragma unroll
+        for (int i = 0; i < V; ++i) sq += keep[k][i] * keep[k][i];
+      }
+    }
+  } else {
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+      gated(c, keep[0]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) sq += keep[0][i] * keep[0][i];
+    }
   }
   for (int off = 16; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
@@ -210,12 +269,17 @@ __global__ void __launch_bounds__(256) ssd_norm_kernel(SsdArgs a) {
   float total = 0.f;
   for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) total += red[w];
   const float inv = rsqrtf(total / width + a.eps);
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
-    float f[V];
-    load_v<V>(v + c, f);
+  if (NV) {
 #pragma unroll
-    for (int i = 0; i < V; ++i) f[i] *= inv * a.norm_w[c0 + c + i];
-    store_v<V>(out + c, f);
+    for (int k = 0; k < NV; ++k) {
+      const int c = (k * blockDim.x + threadIdx.x) * V;
+      if (c < width) write(c, keep[k], inv);
+    }
+  } else {
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+      gated(c, keep[0]);
+      write(c, keep[0], inv);
+    }
   }
   if (blockIdx.y == 0) {
     T* whole = static_cast<T*>(a.out) + row * a.out_ld;
@@ -227,13 +291,13 @@ constexpr int kSdThreads = 256;
 
 // V = 4: vdim is a multiple of 4; V = 1: any vdim.
 template <typename T, int V>
-__global__ void __launch_bounds__(kSdThreads) ssd_decode_kernel(SsdArgs a) {
+__global__ void __launch_bounds__(kSdThreads, 4) ssd_decode_kernel(SsdArgs a) {
   extern __shared__ float sm[];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const int P = a.vdim, N = a.state, inner = a.heads * P, channels = ssd_channels(a);
-  T* vout = static_cast<T*>(a.v) + static_cast<int64_t>(b) * inner + h * P;
+  T* yout = static_cast<T*>(a.y) + static_cast<int64_t>(b) * inner + h * P;
   if (ssd_inactive(a, b)) {
-    for (int c = tid; c < P; c += kSdThreads) vout[c] = T(0.f);
+    for (int c = tid; c < P; c += kSdThreads) yout[c] = T(0.f);
     return;
   }
   const int nc = (P + V - 1) / V;
@@ -256,7 +320,7 @@ __global__ void __launch_bounds__(kSdThreads) ssd_decode_kernel(SsdArgs a) {
   float* s_c = s_b + N;   // [N]
   float* s_o = s_c + N;   // [row groups][P]
   const T* row = static_cast<const T*>(a.proj) + static_cast<int64_t>(b) * a.ld;
-  const int pos = a.start[b], group = h / (a.heads / a.groups);
+  const int pos = a.start[b], here = pos % a.taps, group = h / (a.heads / a.groups);
   const bool owns_bc = h % (a.heads / a.groups) == 0;
   T* ring = static_cast<T*>(a.ring) + static_cast<int64_t>(b) * a.taps * channels;
   const float dt = softplus_f(sf(row[a.dt_off + h]) + a.dt_bias[h]);
@@ -265,11 +329,12 @@ __global__ void __launch_bounds__(kSdThreads) ssd_decode_kernel(SsdArgs a) {
     const int c = i < P ? h * P + i : (i < P + N ? inner + group * N + i - P : inner + a.groups * N + group * N + i - P - N);
     const T cur = row[a.xbc_off + c];
     float acc = a.conv_b[c] + a.conv_w[static_cast<int64_t>(a.taps - 1) * channels + c] * sf(cur);
-    for (int j = 1; j < a.taps && j <= pos; ++j)
-      acc += a.conv_w[static_cast<int64_t>(a.taps - 1 - j) * channels + c] *
-             sf(ring[static_cast<int64_t>((pos - j) % a.taps) * channels + c]);
-    if (i < P || owns_bc) ring[static_cast<int64_t>(pos % a.taps) * channels + c] = cur;
-    acc = silu_f(acc);
+    for (int j = 1, slot = here; j < a.taps && j <= pos; ++j) {
+      slot = slot == 0 ? a.taps - 1 : slot - 1;
+      acc += a.conv_w[static_cast<int64_t>(a.taps - 1 - j) * channels + c] * sf(ring[static_cast<int64_t>(slot) * channels + c]);
+    }
+    if (i < P || owns_bc) ring[static_cast<int64_t>(here) * channels + c] = cur;
+    acc = silu_t(acc, T(0.f));
     sm[i] = i >= P && i < P + N ? acc * dt : acc;
   }
   __syncthreads();
@@ -314,7 +379,7 @@ __global__ void __launch_bounds__(kSdThreads) ssd_decode_kernel(SsdArgs a) {
   for (int p = tid; p < P; p += kSdThreads) {
     float y = a.d[h] * s_x[p];
     for (int g = 0; g < groups; ++g) y += s_o[g * P + p];
-    vout[p] = T(y * silu_f(sf(row[a.z_off + h * P + p])));
+    yout[p] = T(y);
   }
 }
 
@@ -345,7 +410,7 @@ __global__ void __launch_bounds__(kSsThreads) ssd_scan_kernel(SsdArgs a) {
   }
   const T* xbc = static_cast<const T*>(a.xbc) + static_cast<int64_t>(b) * a.T * a.xbc_ld;
   const T* proj = static_cast<const T*>(a.proj) + static_cast<int64_t>(b) * a.T * a.ld;
-  T* vout = static_cast<T*>(a.v) + static_cast<int64_t>(b) * a.T * inner + h * P;
+  T* yout = static_cast<T*>(a.y) + static_cast<int64_t>(b) * a.T * inner + h * P;
   const float rate = -expf(a.a_log[h]), skip = a.d[h];
   for (int t0 = 0; t0 < live; t0 += kSsTok) {
     const int n_tok = min(kSsTok, live - t0);
@@ -387,13 +452,12 @@ __global__ void __launch_bounds__(kSsThreads) ssd_scan_kernel(SsdArgs a) {
       float y = skip * s_x[i];
 #pragma unroll
       for (int g = 0; g < RG; ++g) y += s_o[(t * RG + g) * kSsCols + c];
-      const float z = sf(proj[(t0 + t) * a.ld + a.z_off + h * P + p0 + c]);
-      vout[static_cast<int64_t>(t0 + t) * inner + p0 + c] = T(y * silu_f(z));
+      yout[static_cast<int64_t>(t0 + t) * inner + p0 + c] = T(y);
     }
   }
   for (int i = tid; i < (a.T - live) * kSsCols; i += kSsThreads) {
     const int c = i % kSsCols;
-    if (p0 + c < P) vout[static_cast<int64_t>(live + i / kSsCols) * inner + p0 + c] = T(0.f);
+    if (p0 + c < P) yout[static_cast<int64_t>(live + i / kSsCols) * inner + p0 + c] = T(0.f);
   }
   if (live <= 0) return;
 #pragma unroll
@@ -411,11 +475,11 @@ __global__ void __launch_bounds__(kSsThreads) ssd_scan_kernel(SsdArgs a) {
 //   y_i   = exp(G_i) S_in^T C_i + sum_{j <= i} (C_i . B_j) exp(G_i - G_j) dt_j x_j
 //   S_out = exp(G_63) S_in + sum_j exp(G_63 - G_j) dt_j B_j x_j^T
 //
-// The products C_i . B_j belong to a GROUP, so a CTA takes four units of 16 value columns of one group's
-// heads (one warp each, of the same or of different heads) and computes them once.  Every warp then forms
-// its head's weights in registers.  For a tile of 16 x 16 pairs below the diagonal the decay splits at the
-// end r of the token tile ahead of i's: exp(G_i - G_r) exp(G_r - G_j), both at most one, so no decay strength
-// overflows and the exponentials are per token, not per pair; on the diagonal it is formed per pair.
+// One CTA = 4 warps per (64 value columns of a head, sequence, segment of the prompt).  The pair weights of a
+// 16 x 16 tile come out of one warp's accumulators; below the diagonal their decay splits at the end r of the
+// token tile ahead of i's: exp(G_i - G_r) exp(G_r - G_j), both at most one, so no decay strength overflows and
+// the exponentials are per token, not per pair; on the diagonal they are formed per pair (which also takes the
+// skip d x_i).  Everything else is split by value columns, 16 per warp.
 //
 // What enters the recurrence is kept to fp32 accuracy: pair weights, weighted x and the state as matrix
 // operands are split into two bf16 terms; B, C and x are the bf16 outputs of the convolution.
@@ -428,148 +492,171 @@ __global__ void __launch_bounds__(kSsThreads) ssd_scan_kernel(SsdArgs a) {
 // from its true initial state.
 namespace {
 
-constexpr int kScTok = 64, kScThreads = 128, kScWarps = 4;
+constexpr int kScTok = 64, kScCols = 64, kScThreads = 128;
 constexpr float kL2e = 1.4426950408889634f;
 
 template <int NP>
 struct ScSmem {
-  static constexpr int kNP = NP + 8, kXP = 24, kCP = 72;
-  static constexpr int kB = 0;                                  // bf16 [64][kNP]
-  static constexpr int kC = kB + kScTok * kNP * 2;              // bf16 [64][kNP]
-  static constexpr int kX = kC + kScTok * kNP * 2;              // bf16 [4][64][kXP]
-  static constexpr int kCB = kX + kScWarps * kScTok * kXP * 2;  // float [64][kCP]
-  static constexpr int kG = kCB + kScTok * kCP * 4;             // float [4][64] running log2 decay
-  static constexpr int kDt = kG + kScWarps * kScTok * 4;        // float [4][64]
-  static constexpr int kF = kDt + kScWarps * kScTok * 4;        // float [4][4][64]: dt_j exp(G_(16 r + 15) - G_j)
-  static constexpr int kTotal = kF + kScWarps * 4 * kScTok * 4;
+  static constexpr int kNP = NP + 8, kXP = kScCols + 8;
+  static constexpr int kB = 0;                             // bf16 [64][kNP]
+  static constexpr int kC = kB + kScTok * kNP * 2;         // bf16 [64][kNP]
+  static constexpr int kX = kC + kScTok * kNP * 2;         // bf16 [64][kXP]  x, then y
+  static constexpr int kM = kX + kScTok * kXP * 2;         // bf16 [10 tiles][hi, lo][16][16]  pair weights
+  static constexpr int kG = kM + 10 * 2 * 512;             // float [64] running log2 decay
+  static constexpr int kDt = kG + kScTok * 4;              // float [64]
+  static constexpr int kW = kDt + kScTok * 4;              // float [64]  dt_j exp(G_63 - G_j)
+  static constexpr int kTotal = kW + kScTok * 4;
 };
+
+// S = exp(G_63) S + (w x)^T B with w_j = dt_j exp(G_63 - G_j), hi and lo; ax: x as A fragments (rows = value
+// columns).
+template <int NT>
+__device__ __forceinline__ void update_state(float (&S)[NT][4], const uint32_t (&ax)[4][4], const __nv_bfloat16* sB,
+                                             int pitch, const float* sG, const float* sW, int lane) {
+  const int lc = (lane & 3) * 2;
+  const float end = ex2(sG[kScTok - 1]);
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) S[n][e] *= end;
+#pragma unroll
+  for (int kk = 0; kk < 4; ++kk) {
+    uint32_t ah[4], al[4];
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const float2 w = *reinterpret_cast<const float2*>(sW + kk * 16 + q * 8 + lc);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float2 x = unpack2(ax[kk][2 * q + u]);
+        split2(x.x * w.x, x.y * w.y, ah[2 * q + u], al[2 * q + u]);
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < NT; n += 4) {
+      uint32_t b0[4], b1[4];
+      const __nv_bfloat16* p = sB + (kk * 16 + (lane & 15)) * pitch + n * 8 + (lane >> 4) * 8;
+      ldsm4t(b0, p);
+      ldsm4t(b1, p + 16);
+      mma(S[n], ah, b0[0], b0[1]);
+      mma(S[n + 1], ah, b0[2], b0[3]);
+      mma(S[n + 2], ah, b1[0], b1[1]);
+      mma(S[n + 3], ah, b1[2], b1[3]);
+      mma(S[n], al, b0[0], b0[1]);
+      mma(S[n + 1], al, b0[2], b0[3]);
+      mma(S[n + 2], al, b1[0], b1[1]);
+      mma(S[n + 3], al, b1[2], b1[3]);
+    }
+  }
+}
 
 }  // namespace
 
 template <int NP, bool kStateOnly>
-__global__ void __launch_bounds__(kScThreads, 3) ssd_chunk_kernel(SsdArgs a) {
+__global__ void __launch_bounds__(kScThreads, 4) ssd_chunk_kernel(SsdArgs a) {
   using L = ScSmem<NP>;
   using bf16 = __nv_bfloat16;
   constexpr int NT = NP / 8;
   extern __shared__ __align__(16) uint8_t ssd_smem[];
   bf16* sB = reinterpret_cast<bf16*>(ssd_smem + L::kB);
   bf16* sC = reinterpret_cast<bf16*>(ssd_smem + L::kC);
-  float* sCB = reinterpret_cast<float*>(ssd_smem + L::kCB);
+  bf16* sX = reinterpret_cast<bf16*>(ssd_smem + L::kX);
+  uint8_t* sM = ssd_smem + L::kM;  // the 16-byte halves of a tile's rows swap places every four rows
+  float* sG = reinterpret_cast<float*>(ssd_smem + L::kG);
+  float* sDt = reinterpret_cast<float*>(ssd_smem + L::kDt);
+  float* sW = reinterpret_cast<float*>(ssd_smem + L::kW);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = (lane & 3) * 2;
-  bf16* sX = reinterpret_cast<bf16*>(ssd_smem + L::kX) + warp * kScTok * L::kXP;
-  float* sG = reinterpret_cast<float*>(ssd_smem + L::kG) + warp * kScTok;
-  float* sDt = reinterpret_cast<float*>(ssd_smem + L::kDt) + warp * kScTok;
-  float* sF = reinterpret_cast<float*>(ssd_smem + L::kF) + warp * 4 * kScTok;
 
-  const int P = a.vdim, N = a.state, inner = a.heads * P, hpg = a.heads / a.groups, pt = (P + 15) / 16;
-  const int tiles = (hpg * pt + kScWarps - 1) / kScWarps;
-  const int seg = blockIdx.x, group = blockIdx.y / tiles, b = blockIdx.z;
-  const int unit = (blockIdx.y % tiles) * kScWarps + warp;
-  const bool owner = unit < hpg * pt;
-  const int h = group * hpg + (owner ? unit / pt : 0), p0 = owner ? (unit % pt) * 16 : 0;
-  const int pcols = owner ? min(16, P - p0) : 0;
+  const int P = a.vdim, N = a.state, inner = a.heads * P, blocks = (P + kScCols - 1) / kScCols;
+  const int seg = blockIdx.x, h = blockIdx.y / blocks, p0 = (blockIdx.y % blocks) * kScCols, b = blockIdx.z;
+  const int cols = min(kScCols, P - p0);                  // value columns of this CTA
+  const int v0 = warp * 16, pcols = min(16, cols - v0);   // and of this warp (may be none)
+  const int group = h / (a.heads / a.groups);
   const bool inactive = ssd_inactive(a, b);
   const int live = inactive ? 0 : ssd_live(a, b);
   const int t_lo = seg * a.seg_tokens, t_hi = a.segments > 1 ? min(a.T, t_lo + a.seg_tokens) : a.T;
+  const int t_live = min(live, t_hi);
   const bf16* xbc = static_cast<const bf16*>(a.xbc) + static_cast<int64_t>(b) * a.T * a.xbc_ld;
-  const bf16* proj = static_cast<const bf16*>(a.proj) + static_cast<int64_t>(b) * a.T * a.ld;
-  bf16* vout = static_cast<bf16*>(a.v) + static_cast<int64_t>(b) * a.T * inner + h * P + p0;
-  const int b_off = inner + group * N, c_off = b_off + a.groups * N;
-  const bool vec_bc = !((a.xbc_ld | b_off | c_off | N) & 7), vec_x = !((a.xbc_ld | P) & 7);
-  const bool pairs = !((P | a.z_off | a.ld | inner) & 1);
-  const float rate = owner ? -expf(a.a_log[h]) * kL2e : 0.f, dt_bias = owner ? a.dt_bias[h] : 0.f;
-  const float skip = owner ? a.d[h] : 0.f;
+  const bf16* dt_col = static_cast<const bf16*>(a.proj) + static_cast<int64_t>(b) * a.T * a.ld + a.dt_off + h;
+  bf16* yout = static_cast<bf16*>(a.y) + static_cast<int64_t>(b) * a.T * inner + h * P + p0;
+  const int x_off = h * P + p0, b_off = inner + group * N, c_off = b_off + a.groups * N;
+  const bool vec_bc = !((a.xbc_ld | b_off | c_off | N) & 7), vec_x = !((a.xbc_ld | P | inner) & 7);
+  const float rate = -expf(a.a_log[h]) * kL2e, dt_bias = a.dt_bias[h], skip = a.d[h];
 
   // State, transposed: row = value column, column = state channel.
   float S[NT][4];
   const bool segmented = a.segments > 1;
-  float* state = a.ssm + (static_cast<int64_t>(b) * a.heads + h) * N * P;
+  float* state = a.ssm + (static_cast<int64_t>(b) * a.heads + h) * N * P + p0 + v0;
   float* seg_state =
-      segmented ? a.seg_state + ((static_cast<int64_t>(b) * a.heads + h) * a.segments + seg) * N * P : nullptr;
+      segmented ? a.seg_state + ((static_cast<int64_t>(b) * a.heads + h) * a.segments + seg) * N * P + p0 + v0 : nullptr;
   const float* init = segmented ? seg_state : state;
 #pragma unroll
   for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int p = lr + (e >> 1) * 8, c = n * 8 + lc + (e & 1);
-      S[n][e] = !kStateOnly && p < pcols && c < N ? init[static_cast<int64_t>(c) * P + p0 + p] : 0.f;
+      S[n][e] = !kStateOnly && p < pcols && c < N ? init[static_cast<int64_t>(c) * P + p] : 0.f;
     }
   float decay_sum = 0.f;
+  // Step sizes of the coming chunk (warp 0: tokens lane and lane + 32).
+  float raw[2] = {0.f, 0.f};
+  auto fetch_dt = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (t0 + lane + 32 * i < t_live) raw[i] = __bfloat162float(dt_col[static_cast<int64_t>(t0 + lane + 32 * i) * a.ld]);
+  };
+  if (warp == 0) fetch_dt(t_lo);
 
   for (int t0 = t_lo; t0 < t_hi; t0 += kScTok) {
-    const int rows = max(0, min(kScTok, min(live, t_hi) - t0));
+    const int rows = max(0, min(kScTok, t_live - t0)), n_out = min(kScTok, t_hi - t0);
     if (rows == 0) {  // nothing live here or later in this segment: zero the outputs
-      if (!kStateOnly) {
-        const int n = min(kScTok, t_hi - t0);
-        for (int i = lane; i < n * 16; i += 32)
-          if (i % 16 < pcols) vout[static_cast<int64_t>(t0 + i / 16) * inner + i % 16] = __float2bfloat16(0.f);
-      }
+      if (!kStateOnly)
+        for (int i = tid; i < n_out * kScCols; i += kScThreads)
+          if (i % kScCols < cols) yout[static_cast<int64_t>(t0 + i / kScCols) * inner + i % kScCols] = __float2bfloat16(0.f);
       continue;
     }
     __syncthreads();  // everybody is done with the previous chunk's tiles
     const bf16* src = xbc + static_cast<int64_t>(t0) * a.xbc_ld;
-    auto load_bc = [&](bf16* tile, int off) {
-      constexpr int kPer = NP / 8, kStep = kScThreads / kPer;
-      const int c = (tid % kPer) * 8;
+    // `width` columns of the chunk's rows into a tile of W columns, zero beyond.
+    auto load_tile = [&](auto w_const, bf16* tile, int pitch, int off, int width, bool vec) {
+      constexpr int W = decltype(w_const)::value, kPer = W / 8, kStep = kScThreads / kPer;
+      const int c = (tid % kPer) * 8, r0 = tid / kPer;
+      bf16* dst = tile + r0 * pitch + c;
+      const bf16* p = src + r0 * a.xbc_ld + off + c;
+      if (vec && c < width && rows == kScTok) {
 #pragma unroll
-      for (int r = tid / kPer; r < kScTok; r += kStep) {
-        bf16* dst = tile + r * L::kNP + c;
-        const bf16* p = src + r * a.xbc_ld + off + c;
-        if (vec_bc && r < rows && c < N) {
-          cp16(dst, p);
-        } else if (vec_bc || r >= rows || c >= N) {
+        for (int i = 0; i < kScTok / kStep; ++i) {
+          cp16(dst + i * kStep * pitch, p);
+          p += kStep * a.xbc_ld;
+        }
+        return;
+      }
+#pragma unroll 1
+      for (int r = r0; r < kScTok; r += kStep) {
+        if (r >= rows || c >= width) {
           *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        } else if (vec) {
+          cp16(dst, p);
         } else {
 #pragma unroll 1
-          for (int e = 0; e < 8; ++e) dst[e] = c + e < N ? p[e] : __float2bfloat16(0.f);
+          for (int e = 0; e < 8; ++e) dst[e] = c + e < width ? p[e] : __float2bfloat16(0.f);
         }
+        dst += kStep * pitch;
+        p += kStep * a.xbc_ld;
       }
     };
-    load_bc(sB, b_off);
-    if (!kStateOnly) load_bc(sC, c_off);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {  // the warp's own 64 x 16 slice of x
-      const int r = i * 16 + (lane >> 1), c = (lane & 1) * 8;
-      bf16* dst = sX + r * L::kXP + c;
-      const bf16* p = src + r * a.xbc_ld + h * P + p0 + c;
-      if (vec_x && r < rows && c < pcols) {
-        cp16(dst, p);
-      } else if (vec_x || r >= rows || c >= pcols) {
-        *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-      } else {
-#pragma unroll 1
-        for (int e = 0; e < 8; ++e) dst[e] = c + e < pcols ? p[e] : __float2bfloat16(0.f);
-      }
-    }
+    load_tile(std::integral_constant<int, NP>(), sB, L::kNP, b_off, N, vec_bc);
+    if (!kStateOnly) load_tile(std::integral_constant<int, NP>(), sC, L::kNP, c_off, N, vec_bc);
+    load_tile(std::integral_constant<int, kScCols>(), sX, L::kXP, x_off, cols, vec_x);
     cp_commit();
+    // The next chunk's x starts its way from DRAM to L2 (B and C are shared by the heads of a group).
+    if (tid >= 64 && t0 + tid < t_live) asm volatile("prefetch.global.L2 [%0];" ::"l"(src + tid * a.xbc_ld + x_off));
 
-    // Gates of this warp's outputs (rows lr + 8 k), as bf16 pairs.
-    uint32_t z[8][2];
-    if (!kStateOnly) {
-#pragma unroll
-      for (int m = 0; m < 8; ++m)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const int r = m * 8 + lr, c = n * 8 + lc;
-          z[m][n] = 0;
-          if (r < rows && c < pcols) {
-            const bf16* p = proj + (t0 + r) * a.ld + a.z_off + h * P + p0 + c;
-            if (pairs) {
-              z[m][n] = *reinterpret_cast<const uint32_t*>(p);
-            } else {
-              __nv_bfloat162 q = __halves2bfloat162(p[0], c + 1 < pcols ? p[1] : p[0]);
-              z[m][n] = reinterpret_cast<uint32_t&>(q);
-            }
-          }
-        }
-    }
-    // Step sizes and running log decays of the warp's head: lane holds tokens lane and lane + 32.
-    {
+    if (warp == 0) {
+      // Step sizes and running log decays.
       float dt[2], g[2];
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
-        const int r = lane + 32 * i;
-        dt[i] = owner && r < rows ? softplus_f(__bfloat162float(proj[(t0 + r) * a.ld + a.dt_off + h]) + dt_bias) : 0.f;
+        dt[i] = lane + 32 * i < rows ? softplus_f(raw[i] + dt_bias) : 0.f;
         g[i] = rate * dt[i];
 #pragma unroll
         for (int off = 1; off < 32; off <<= 1) {
@@ -578,49 +665,79 @@ __global__ void __launch_bounds__(kScThreads, 3) ssd_chunk_kernel(SsdArgs a) {
         }
       }
       g[1] += __shfl_sync(0xffffffffu, g[0], 31);
-      const float ref[4] = {__shfl_sync(0xffffffffu, g[0], 15), __shfl_sync(0xffffffffu, g[0], 31),
-                            __shfl_sync(0xffffffffu, g[1], 15), __shfl_sync(0xffffffffu, g[1], 31)};
-      decay_sum += ref[3];
+      const float end = __shfl_sync(0xffffffffu, g[1], 31);
+      decay_sum += end;
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
-        const int r = lane + 32 * i;
-        sG[r] = g[i];
-        sDt[r] = dt[i];
-#pragma unroll
-        for (int q = kStateOnly ? 3 : 0; q < 4; ++q) sF[q * kScTok + r] = r < 16 * (q + 1) ? dt[i] * ex2(ref[q] - g[i]) : 0.f;
+        sG[lane + 32 * i] = g[i];
+        sDt[lane + 32 * i] = dt[i];
+        sW[lane + 32 * i] = dt[i] * ex2(end - g[i]);
       }
+      fetch_dt(t0 + kScTok);
     }
     cp_wait_all();
     __syncthreads();
 
-    float O[4][2][4];
     if (!kStateOnly) {
-      // Products C_i . B_j of the ten 16 x 16 tiles on and below the diagonal, shared out over the warps.
-      for (int tile = warp; tile < 10; tile += kScWarps) {
-        const int m = tile < 1 ? 0 : tile < 3 ? 1 : tile < 6 ? 2 : 3, n = tile - m * (m + 1) / 2;
-        float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      // Weights of the ten 16 x 16 tiles of pairs on and below the diagonal: a diagonal tile per warp, then the
+      // other six.
+#pragma unroll 1
+      for (int tile = warp; tile < 10; tile += 4) {
+        const int q = tile - 4;  // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
+        const int m = tile < 4 ? tile : q < 1 ? 1 : q < 3 ? 2 : 3, n = tile < 4 ? tile : q - m * (m - 1) / 2;
+        float s[2][4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[u][e] = 0.f;
 #pragma unroll
         for (int k = 0; k < NP; k += 16) {
           uint32_t af[4], bf[4];
           ldsm4(af, sC + (m * 16 + (lane & 15)) * L::kNP + k + (lane >> 4) * 8);
           ldsm4(bf, sB + (n * 16 + (lane >> 4) * 8 + (lane & 7)) * L::kNP + k + ((lane >> 3) & 1) * 8);
-          mma(c0, af, bf[0], bf[1]);
-          mma(c1, af, bf[2], bf[3]);
+          mma(s[0], af, bf[0], bf[1]);
+          mma(s[1], af, bf[2], bf[3]);
         }
+        const int r0 = m * 16 + lr, r1 = r0 + 8;
+        const float g0 = sG[r0], g1 = sG[r1];
+        const float ref = sG[max(m * 16 - 1, 0)];
+        const float d0 = ex2(g0 - ref), d1 = ex2(g1 - ref);  // off the diagonal
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          float* dst = sCB + (m * 16 + lr + half * 8) * L::kCP + n * 16 + lc;
-          *reinterpret_cast<float2*>(dst) = make_float2(c0[half * 2], c0[half * 2 + 1]);
-          *reinterpret_cast<float2*>(dst + 8) = make_float2(c1[half * 2], c1[half * 2 + 1]);
+        for (int u = 0; u < 2; ++u) {
+          const int c = n * 16 + u * 8 + lc;
+          const float2 g = *reinterpret_cast<const float2*>(sG + c), dt = *reinterpret_cast<const float2*>(sDt + c);
+          float w[4];
+          if (tile >= 4) {
+            const float fx = dt.x * ex2(ref - g.x), fy = dt.y * ex2(ref - g.y);
+            w[0] = s[u][0] * d0 * fx, w[1] = s[u][1] * d0 * fy, w[2] = s[u][2] * d1 * fx, w[3] = s[u][3] * d1 * fy;
+          } else {
+            w[0] = c <= r0 ? s[u][0] * ex2(g0 - g.x) * dt.x : 0.f;
+            w[1] = c + 1 <= r0 ? s[u][1] * ex2(g0 - g.y) * dt.y : 0.f;
+            w[2] = c <= r1 ? s[u][2] * ex2(g1 - g.x) * dt.x : 0.f;
+            w[3] = c + 1 <= r1 ? s[u][3] * ex2(g1 - g.y) * dt.y : 0.f;
+            if (c == r0) w[0] += skip;
+            if (c + 1 == r0) w[1] += skip;
+            if (c == r1) w[2] += skip;
+            if (c + 1 == r1) w[3] += skip;
+          }
+          uint32_t hi, lo;
+          uint8_t* at = sM + (m * (m + 1) / 2 + n) * 1024 + lr * 32 + (u ^ (lr >> 2 & 1)) * 16 + lc * 2;
+          split2(w[0], w[1], hi, lo);
+          *reinterpret_cast<uint32_t*>(at) = hi;
+          *reinterpret_cast<uint32_t*>(at + 512) = lo;
+          split2(w[2], w[3], hi, lo);
+          *reinterpret_cast<uint32_t*>(at + 256) = hi;
+          *reinterpret_cast<uint32_t*>(at + 768) = lo;
         }
       }
+      // O = C S_in: the state's accumulators as B fragments, hi and lo.
+      float O[4][2][4];
 #pragma unroll
       for (int m = 0; m < 4; ++m)
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e) O[m][n][e] = 0.f;
-      // O = C S_in: the state's accumulators as B fragments, hi and lo.
 #pragma unroll
       for (int kk = 0; kk < NP / 16; ++kk) {
         uint32_t bh[2][2], bl[2][2];
@@ -633,107 +750,74 @@ __global__ void __launch_bounds__(kScThreads, 3) ssd_chunk_kernel(SsdArgs a) {
           uint32_t af[4];
           ldsm4(af, sC + (m * 16 + (lane & 15)) * L::kNP + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            mma(O[m][u], af, bh[u][0], bh[u][1]);
-            mma(O[m][u], af, bl[u][0], bl[u][1]);
-          }
+          for (int u = 0; u < 2; ++u) mma(O[m][u], af, bh[u][0], bh[u][1]);
+#pragma unroll
+          for (int u = 0; u < 2; ++u) mma(O[m][u], af, bl[u][0], bl[u][1]);
         }
       }
-      __syncthreads();  // all products are in shared memory
-      uint32_t bx[4][4];
-#pragma unroll
-      for (int kk = 0; kk < 4; ++kk) ldsm4t(bx[kk], sX + (kk * 16 + (lane & 15)) * L::kXP + (lane >> 4) * 8);
 #pragma unroll
       for (int m = 0; m < 4; ++m) {
-        const int r0 = m * 16 + lr, r1 = r0 + 8;
-        const float g0 = sG[r0], g1 = sG[r1];
-        const float e0 = ex2(g0), e1 = ex2(g1);
+        const float e0 = ex2(sG[m * 16 + lr]), e1 = ex2(sG[m * 16 + lr + 8]);
 #pragma unroll
         for (int n = 0; n < 2; ++n) O[m][n][0] *= e0, O[m][n][1] *= e0, O[m][n][2] *= e1, O[m][n][3] *= e1;
-        const float ref = m > 0 ? sG[m > 0 ? m * 16 - 1 : 0] : 0.f;
-        const float d0 = ex2(g0 - ref), d1 = ex2(g1 - ref);
-#pragma unroll
-        for (int kk = 0; kk <= m; ++kk) {
-          uint32_t ah[4], al[4];
-#pragma unroll
-          for (int q = 0; q < 2; ++q) {  // columns kk * 16 + q * 8 + lc, + 1
-            const int c = kk * 16 + q * 8 + lc;
-            const float2 s0 = *reinterpret_cast<const float2*>(sCB + r0 * L::kCP + c);
-            const float2 s1 = *reinterpret_cast<const float2*>(sCB + r1 * L::kCP + c);
-            float2 w0, w1;
-            if (kk < m) {
-              const float2 f = *reinterpret_cast<const float2*>(sF + (m > 0 ? m - 1 : 0) * kScTok + c);
-              w0 = make_float2(d0 * f.x, d0 * f.y), w1 = make_float2(d1 * f.x, d1 * f.y);
-            } else {
-              const float2 g = *reinterpret_cast<const float2*>(sG + c), dt = *reinterpret_cast<const float2*>(sDt + c);
-              w0 = make_float2(c <= r0 ? ex2(g0 - g.x) * dt.x : 0.f, c + 1 <= r0 ? ex2(g0 - g.y) * dt.y : 0.f);
-              w1 = make_float2(c <= r1 ? ex2(g1 - g.x) * dt.x : 0.f, c + 1 <= r1 ? ex2(g1 - g.y) * dt.y : 0.f);
-            }
-            split2(s0.x * w0.x, s0.y * w0.y, ah[2 * q], al[2 * q]);
-            split2(s1.x * w1.x, s1.y * w1.y, ah[2 * q + 1], al[2 * q + 1]);
-          }
-#pragma unroll
-          for (int n = 0; n < 2; ++n) {
-            mma(O[m][n], ah, bx[kk][2 * n], bx[kk][2 * n + 1]);
-            mma(O[m][n], al, bx[kk][2 * n], bx[kk][2 * n + 1]);
-          }
-        }
       }
-    }
-    // S = exp(G_63) S + (w x)^T B with w_j = dt_j exp(G_63 - G_j), hi and lo.
-    {
-      const float end = ex2(sG[kScTok - 1]);
-#pragma unroll
-      for (int n = 0; n < NT; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[n][e] *= end;
+      __syncthreads();  // all weights are in shared memory
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
-        uint32_t ax[4], ah[4], al[4];
-        ldsm4t(ax, sX + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * L::kXP + ((lane >> 3) & 1) * 8);
+        uint32_t bx[4];
+        ldsm4t(bx, sX + (kk * 16 + (lane & 15)) * L::kXP + v0 + (lane >> 4) * 8);
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          const float2 w = *reinterpret_cast<const float2*>(sF + 3 * kScTok + kk * 16 + q * 8 + lc);
-#pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            const float2 x = unpack2(ax[2 * q + u]);
-            split2(x.x * w.x, x.y * w.y, ah[2 * q + u], al[2 * q + u]);
-          }
-        }
-#pragma unroll
-        for (int n = 0; n < NT; n += 2) {
-          uint32_t bf[4];
-          ldsm4t(bf, sB + (kk * 16 + (lane & 15)) * L::kNP + n * 8 + (lane >> 4) * 8);
-          mma(S[n], ah, bf[0], bf[1]);
-          mma(S[n + 1], ah, bf[2], bf[3]);
-          mma(S[n], al, bf[0], bf[1]);
-          mma(S[n + 1], al, bf[2], bf[3]);
+        for (int m = kk; m < 4; ++m) {
+          uint32_t ah[4], al[4];
+          const uint8_t* at = sM + (m * (m + 1) / 2 + kk) * 1024 + (lane & 15) * 32 + ((lane >> 4) ^ (lane >> 2 & 1)) * 16;
+          ldsm4(ah, at);
+          ldsm4(al, at + 512);
+          mma(O[m][0], ah, bx[0], bx[1]);
+          mma(O[m][1], ah, bx[2], bx[3]);
+          mma(O[m][0], al, bx[0], bx[1]);
+          mma(O[m][1], al, bx[2], bx[3]);
         }
       }
+      // The state's update reads x once more; y then takes its place (the warp's own columns).
+      uint32_t ax[4][4];
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk)
+        ldsm4t(ax[kk], sX + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * L::kXP + v0 + ((lane >> 3) & 1) * 8);
+      __syncwarp();
+#pragma unroll
+      for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const int r = m * 16 + lr + half * 8;
+            *reinterpret_cast<uint32_t*>(sX + r * L::kXP + v0 + n * 8 + lc) =
+                r < rows ? pack2(O[m][n][half * 2], O[m][n][half * 2 + 1]) : 0u;
+          }
+      __syncwarp();
+      update_state<NT>(S, ax, sB, L::kNP, sG, sW, lane);
+      if (vec_x) {
+        const int c = (lane & 1) * 8;
+        if (c < pcols) {
+          bf16* dst = yout + static_cast<int64_t>(t0 + (lane >> 1)) * inner + v0 + c;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int r = i * 16 + (lane >> 1);
+            if (r < n_out) *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(sX + r * L::kXP + v0 + c);
+            dst += static_cast<int64_t>(16) * inner;
+          }
+        }
+      } else {
+        for (int i = lane; i < n_out * 16; i += 32)
+          if (i % 16 < pcols) yout[static_cast<int64_t>(t0 + i / 16) * inner + v0 + i % 16] = sX[i / 16 * L::kXP + v0 + i % 16];
+      }
+    } else {
+      uint32_t ax[4][4];
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk)
+        ldsm4t(ax[kk], sX + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * L::kXP + v0 + ((lane >> 3) & 1) * 8);
+      update_state<NT>(S, ax, sB, L::kNP, sG, sW, lane);
     }
-    if (kStateOnly) continue;
-    const int n_out = min(kScTok, t_hi - t0);
-#pragma unroll
-    for (int m = 0; m < 8; ++m)
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        const int r = m * 8 + lr, c = n * 8 + lc;
-        if (r < n_out && c < pcols) {
-          const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(sX + r * L::kXP + c)), g = unpack2(z[m][n]);
-          float y0 = 0.f, y1 = 0.f;
-          if (r < rows) {
-            y0 = (O[m >> 1][n][(m & 1) * 2] + skip * x.x) * __fdividef(g.x, 1.f + ex2(-g.x * kL2e));
-            y1 = (O[m >> 1][n][(m & 1) * 2 + 1] + skip * x.y) * __fdividef(g.y, 1.f + ex2(-g.y * kL2e));
-          }
-          bf16* dst = vout + static_cast<int64_t>(t0 + r) * inner + c;
-          if (pairs) {
-            *reinterpret_cast<uint32_t*>(dst) = pack2(y0, y1);
-          } else {
-            dst[0] = __float2bfloat16(y0);
-            if (c + 1 < pcols) dst[1] = __float2bfloat16(y1);
-          }
-        }
-      }
   }
 
   // Final state: of the sequence (last segment), or of this segment alone.
@@ -745,9 +829,9 @@ __global__ void __launch_bounds__(kScThreads, 3) ssd_chunk_kernel(SsdArgs a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int p = lr + (e >> 1) * 8, c = n * 8 + lc + (e & 1);
-      if (p < pcols && c < N) dst[static_cast<int64_t>(c) * P + p0 + p] = S[n][e];
+      if (p < pcols && c < N) dst[static_cast<int64_t>(c) * P + p] = S[n][e];
     }
-  if (kStateOnly && owner && p0 == 0 && lane == 0)
+  if (kStateOnly && p0 == 0 && tid == 0)
     a.seg_decay[(static_cast<int64_t>(b) * a.heads + h) * a.segments + seg] = decay_sum;
 }
 
@@ -759,11 +843,22 @@ __global__ void ssd_segment_kernel(SsdArgs a) {
   const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= n) return;
   float s = a.ssm[bh * n + i];
-  for (int g = 0; g < a.segments; ++g) {
-    float* p = a.seg_state + (bh * a.segments + g) * n + i;
-    const float add = *p;
-    *p = s;
-    s = s * exp2f(a.seg_decay[bh * a.segments + g]) + add;
+  float* p = a.seg_state + bh * a.segments * n + i;
+  constexpr int kBatch = 8;
+  for (int g0 = 0; g0 < a.segments; g0 += kBatch) {
+    float add[kBatch], decay[kBatch];
+#pragma unroll
+    for (int u = 0; u < kBatch; ++u)
+      if (g0 + u < a.segments) {
+        add[u] = p[(g0 + u) * n];
+        decay[u] = a.seg_decay[bh * a.segments + g0 + u];
+      }
+#pragma unroll
+    for (int u = 0; u < kBatch; ++u)
+      if (g0 + u < a.segments) {
+        p[(g0 + u) * n] = s;
+        s = s * exp2f(decay[u]) + add[u];
+      }
   }
 }
 
@@ -848,9 +943,7 @@ int launch_chunk_pass(const SsdArgs& a, cudaStream_t stream) {
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
     configured = true;
   }
-  const int units = a.heads / a.groups * ((a.vdim + 15) / 16);
-  const int tiles = (units + kScWarps - 1) / kScWarps;
-  kernel<<<dim3(a.segments, a.groups * tiles, a.B), kScThreads, smem, stream>>>(a);
+  kernel<<<dim3(a.segments, a.heads * ((a.vdim + kScCols - 1) / kScCols), a.B), kScThreads, smem, stream>>>(a);
   return launched();
 }
 
@@ -870,14 +963,20 @@ template <typename T>
 int norm(const SsdArgs& a, cudaStream_t stream) {
   const int inner = a.heads * a.vdim, width = inner / a.norm_groups;
   const int64_t rows = static_cast<int64_t>(a.B) * a.T;
-  const bool vec = !((width | inner | static_cast<int>(a.out_ld)) & 7);
+  const bool vec = !((width | inner | a.z_off | static_cast<int>(a.out_ld | a.ld)) & 7);
   const int want = ((vec ? width / 8 : width) + 31) / 32 * 32;
   const int threads = want < 32 ? 32 : (want > 256 ? 256 : want);
   const dim3 grid(static_cast<unsigned>(rows), a.norm_groups);
-  if (vec)
-    ssd_norm_kernel<T, 8><<<grid, threads, 0, stream>>>(a);
+  if (!vec)
+    ssd_norm_kernel<T, 1, 0><<<grid, threads, 0, stream>>>(a);
+  else if (width <= 8 * 256)
+    ssd_norm_kernel<T, 8, 1><<<grid, threads, 0, stream>>>(a);
+  else if (width <= 16 * 256)
+    ssd_norm_kernel<T, 8, 2><<<grid, threads, 0, stream>>>(a);
+  else if (width <= 32 * 256)
+    ssd_norm_kernel<T, 8, 4><<<grid, threads, 0, stream>>>(a);
   else
-    ssd_norm_kernel<T, 1><<<grid, threads, 0, stream>>>(a);
+    ssd_norm_kernel<T, 8, 0><<<grid, threads, 0, stream>>>(a);
   return launched();
 }
 
@@ -891,7 +990,7 @@ extern "C" int axb_ssd_conv(const axb::SsdArgs* args, cudaStream_t stream) {
   return a.act_bf16 ? axb::conv<__nv_bfloat16>(a, stream) : axb::conv<float>(a, stream);
 }
 
-// Gated outputs into a.v, token by token; needs a.xbc.  state <= 512.
+// Outputs into a.y, token by token; needs a.xbc.  state <= 512.
 extern "C" int axb_ssd_scan(const axb::SsdArgs* args, cudaStream_t stream) {
   const axb::SsdArgs& a = *args;
   if (axb::ssd_bad(a) || a.xbc == nullptr || a.state > 512) return -10;

@@ -1,14 +1,16 @@
-"""Serving throughput of Sagisun beside the Fuji decoder of the same widths (one GPU, random weights).
+"""Serving throughput of Sagisun and Zukitar beside the Fuji decoder of the same widths (one GPU, random weights).
 
-Both models run on their decode engines: prompts of equal length, then greedy decoding from a captured
-step.  ``bench.py --serving`` prints one JSON line per (size, model, batch); ``--serving_table FILE`` adds
-the device time of every kernel of one prompt pass and one decoding step.  Layers are identical, so a few
-of them give the per-layer cost; the vocabulary product is included once.
+All models run on their decode engines: prompts of equal length, then greedy decoding from a captured
+step.  ``bench.py --serving`` prints one JSON line per (size, model, batch); ``--serving_models`` picks models,
+``--serving_table FILE`` adds the device time of every kernel of one prompt pass and one decoding step.  Layers
+repeat (Zukitar in threes: two state-space, one latent-attention), so a few of them give the per-layer cost;
+the vocabulary product is included once.
 """
 
 from __future__ import annotations
 
 import collections
+import functools
 import gc
 import json
 from typing import Optional
@@ -16,22 +18,22 @@ from typing import Optional
 import torch
 
 from axlearn_b200.common import prng
-from axlearn_b200.experiments.text.gpt import sagisun
+from axlearn_b200.experiments.text.gpt import sagisun, zukitar
 from axlearn_b200.inference.bench_decode import random_weights
 from axlearn_b200.inference.decode_engine import DecodeEngine, FujiDims, ModuleDecodeEngine
 from axlearn_b200.ops import cuda_ops
 
 # Layers per model and (batch, prompt length, decoding steps) per size.
 SIZES = {
-    "1B": dict(layers=8, runs=[(1, 2048, 64), (8, 2048, 64), (64, 512, 64)]),
-    "7B": dict(layers=4, runs=[(1, 4096, 64), (8, 2048, 64), (64, 512, 64)]),
+    "1B": dict(layers=9, runs=[(1, 2048, 64), (8, 2048, 64), (64, 512, 64)]),
+    "7B": dict(layers=6, runs=[(1, 4096, 64), (8, 2048, 64), (64, 512, 64)]),
 }
 
 
-def _sagisun_engine(size: str, layers: int, batch: int, max_len: int) -> ModuleDecodeEngine:
-    cfg = sagisun.size_config(size)
-    cfg["layers"] = cfg["layers"][:1] * layers
-    model = sagisun.model_config(cfg).set(name="model", dtype=torch.bfloat16).instantiate(parent=None)
+def _module_engine(module, size: str, layers: int, batch: int, max_len: int) -> ModuleDecodeEngine:
+    cfg = module.size_config(size)
+    cfg["layers"] = cfg["layers"][:layers]
+    model = module.model_config(cfg).set(name="model", dtype=torch.bfloat16).instantiate(parent=None)
     params = model.initialize_parameters_recursively(prng.PRNGKey(0), device="cuda")
     return ModuleDecodeEngine(model.decoder, params["decoder"], batch=batch, max_len=max_len, device="cuda")
 
@@ -69,15 +71,21 @@ def _kernel_times(fn) -> list:
         if e.device_type == torch.autograd.DeviceType.CUDA:
             total[e.name[:110]] += e.device_time
             count[e.name[:110]] += 1
-    return [(t, count[n], n) for n, t in total.most_common(16)]
+    return [(t, count[n], n) for n, t in total.most_common(24)]
 
 
-def run(*, steps: int, warmup: int, table: Optional[str] = None, sizes: Optional[list] = None, emit=print) -> list:
+ENGINES = {"zukitar": functools.partial(_module_engine, zukitar), "sagisun": functools.partial(_module_engine, sagisun),
+           "fuji": _fuji_engine}
+
+
+def run(*, steps: int, warmup: int, table: Optional[str] = None, sizes: Optional[list] = None,
+        models: Optional[list] = None, emit=print) -> list:
     results = []
     out = open(table, "w", encoding="utf-8") if table else None
     for size in sizes or list(SIZES):
         spec = SIZES[size]
-        for name, make in (("sagisun", _sagisun_engine), ("fuji", _fuji_engine)):
+        for name in models or list(ENGINES):
+            make = ENGINES[name]
             for batch, prompt, new in spec["runs"]:
                 engine = make(size, spec["layers"], batch, prompt + new + 16)
                 ids = torch.randint(0, engine.logits.shape[1], (batch, prompt),

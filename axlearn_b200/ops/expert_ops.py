@@ -12,6 +12,7 @@ expert; 32-bit runs use the plain kernel of ``csrc/skinny_group.cu``.
 from __future__ import annotations
 
 import ctypes
+import functools
 
 import torch
 
@@ -139,8 +140,9 @@ def _cuda_expert_feed_forward(h, logits, gate_up, down, *, top, width, hidden, g
             return y.reshape(shape[:-1] + (out_ld,))
         place = None
     else:
-        act = gated_act(moe_ops._gmm_kernel(x, gate_up, block_expert, transpose_w=True), half, half, gate)  # pylint: disable=protected-access
-        y = moe_ops._gmm_kernel(act, down, block_expert, transpose_w=True)  # pylint: disable=protected-access
+        # Rows between the runs hold anything; nobody reads their results.
+        product = functools.partial(moe_ops._gmm_kernel, block_expert=block_expert, transpose_w=True, zero_unused=False)  # pylint: disable=protected-access
+        y = product(gated_act(product(x, gate_up), half, half, gate), down)
     out = torch.empty((tokens, out_ld), dtype=h.dtype, device=dev)
     check(lib.axb_expert_combine(y.data_ptr(), None if place is None else place.data_ptr(), out.data_ptr(), tokens,
                                  y.stride(0), out_ld, top, out_ld, int(bf16), stream), "axb_expert_combine")

@@ -154,7 +154,7 @@ class _Args(ctypes.Structure):
     """Mirrors ``axb::LatentArgs``."""
 
     _fields_ = [(n, ctypes.c_void_p) for n in (
-        "proj", "norm_w", "freq", "cache", "lat", "qbuf", "out", "part", "tickets", "start", "live")] + [
+        "proj", "norm_w", "freq", "cache", "lat", "qbuf", "out", "part", "part_ml", "start", "live")] + [
         (n, ctypes.c_int64) for n in ("ld", "cache_ld", "lat_ld", "out_ld")] + [(n, ctypes.c_int) for n in (
             "B", "T", "heads", "dim", "rot_dim", "rot_dims", "rank", "rot_off", "row_w", "slots", "q_off", "c_off",
             "r_off", "splits", "act_bf16")] + [("scale", ctypes.c_float), ("eps", ctypes.c_float)]
@@ -200,8 +200,8 @@ def flash_supported(spec: LatentSpec, proj: Tensor, cols: LatentColumns) -> bool
 
 
 def decode_splits(ctas: int, keys: int, sms: int = 148) -> int:
-    """Cuts of the cached rows in a decoding step: about one CTA per SM, at least 128 keys each."""
-    return max(1, min(sms // max(1, ctas), keys // 128, 64))
+    """Cuts of the cached rows in a decoding step: about one CTA per SM, at least one tile of 64 keys each."""
+    return max(1, min(sms // max(1, ctas), -(-keys // 64), 64))
 
 
 def _cuda_latent_attention(proj, norm_scale, uk, uv, spec, cols, *, start, live, cache, form: Optional[str] = None):
@@ -209,7 +209,7 @@ def _cuda_latent_attention(proj, norm_scale, uk, uv, spec, cols, *, start, live,
     choice."""
     from axlearn_b200 import ops
     from axlearn_b200.ops import cuda_ops, skinny_ops
-    from axlearn_b200.ops.window_ops import _int32, _ticket_buffer
+    from axlearn_b200.ops.window_ops import _int32
 
     lib = _lib()
     proj = proj.contiguous()
@@ -265,11 +265,11 @@ def _cuda_latent_attention(proj, norm_scale, uk, uv, spec, cols, *, start, live,
     lat_out = torch.empty((b * t, h, spec.rot_offset), dtype=proj.dtype, device=proj.device)
     a.out, a.out_ld = lat_out.data_ptr(), spec.rot_offset
     if form != "plain" and proj.dtype == torch.bfloat16 and lib.axb_latent_decode_supported(spec.row_width, spec.rank):
-        ctas = b * t * -(-h // 16)
+        ctas = b * t * -(-h // (32 if h > 16 else 16))
         a.splits = decode_splits(ctas, rows.shape[1])
         if a.splits > 1:
             part = torch.empty(b * t * h * a.splits * (spec.rot_offset + 2), dtype=torch.float32, device=proj.device)
-            a.part, a.tickets = part.data_ptr(), _ticket_buffer(proj.device, ctas).data_ptr()
+            a.part, a.part_ml = part.data_ptr(), part[b * t * h * a.splits * spec.rot_offset:].data_ptr()
         check(lib.axb_latent_decode(ctypes.byref(a), stream), "axb_latent_decode")
     else:
         check(lib.axb_latent_attn(ctypes.byref(a), stream), "axb_latent_attn")

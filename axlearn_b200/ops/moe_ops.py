@@ -199,12 +199,13 @@ def _grouped_argtypes():
     return h
 
 
-def _gmm_kernel(x, w, block_expert, transpose_w: bool):
-    """``out[r] = x[r] @ (w[g(r)]^T if transpose_w else w[g(r)])`` on the tcgen05 kernel."""
+def _gmm_kernel(x, w, block_expert, transpose_w: bool, zero_unused: bool = True):
+    """``out[r] = x[r] @ (w[g(r)]^T if transpose_w else w[g(r)])`` on the tcgen05 kernel.  Rows of unused
+    blocks are zero, or left as they are with ``zero_unused=False``."""
     rows, k = x.shape
     e = w.shape[0]
     n = w.shape[1] if transpose_w else w.shape[2]
-    out = torch.zeros((rows, n), dtype=torch.bfloat16, device=x.device)
+    out = (torch.zeros if zero_unused else torch.empty)((rows, n), dtype=torch.bfloat16, device=x.device)
     rc = _grouped_argtypes().axb_gemm_bf16_grouped(
         x.data_ptr(), w.data_ptr(), out.data_ptr(), rows, n, k, x.stride(0), w.stride(1), out.stride(0),
         0, 0 if transpose_w else 1, 0, 1, e, block_expert.data_ptr(), 0, GROUP_BLOCK,

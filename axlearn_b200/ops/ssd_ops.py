@@ -164,7 +164,7 @@ class _Args(ctypes.Structure):
     """Mirrors ``axb::SsdArgs``."""
 
     _fields_ = [(n, ctypes.c_void_p) for n in (
-        "proj", "conv_w", "conv_b", "dt_bias", "a_log", "d", "norm_w", "ssm", "ring", "xbc", "v", "out",
+        "proj", "conv_w", "conv_b", "dt_bias", "a_log", "d", "norm_w", "ssm", "ring", "xbc", "y", "out",
         "seg_state", "seg_decay", "start", "live")] + [(n, ctypes.c_int64) for n in (
             "ld", "xbc_ld", "out_ld")] + [(n, ctypes.c_int) for n in (
                 "B", "T", "heads", "vdim", "state", "groups", "taps", "norm_groups", "z_off", "xbc_off", "dt_off",
@@ -188,7 +188,7 @@ def _lib():
     return h
 
 
-def prompt_segments(ctas: int, t: int, slots: int = 296) -> tuple[int, int]:
+def prompt_segments(ctas: int, t: int, slots: int = 592) -> tuple[int, int]:
     """``(segments, tokens per segment)`` of a prompt pass that has ``ctas`` independent CTAs per segment: cut
     until ``slots`` of them run at once, no shorter than 256 tokens; a cut costs a second pass over x and B."""
     want = min(slots // max(1, ctas), t // 256)
@@ -199,9 +199,8 @@ def prompt_segments(ctas: int, t: int, slots: int = 296) -> tuple[int, int]:
 
 
 def chunk_ctas(spec: SsdSpec) -> int:
-    """CTAs per sequence of the chunked kernel: four 16-column units of one group's heads each."""
-    units = spec.heads // spec.groups * -(-spec.vdim // 16)
-    return spec.groups * -(-units // 4)
+    """CTAs per sequence of the chunked kernel: 64 value columns of a head each."""
+    return spec.heads * -(-spec.vdim // 64)
 
 
 def _cuda_ssd_mix(proj, w: SsdWeights, spec: SsdSpec, cols: SsdColumns, *, start, live, state,
@@ -240,8 +239,8 @@ def _cuda_ssd_mix(proj, w: SsdWeights, spec: SsdSpec, cols: SsdColumns, *, start
     a.norm_groups, a.eps = spec.norm_groups, spec.eps
     a.z_off, a.xbc_off, a.dt_off = cols.z, cols.xbc, cols.dt
     a.act_bf16, a.segments, a.seg_tokens = int(proj.dtype == torch.bfloat16), 1, padded(t, CHUNK_TOKENS)
-    v = torch.empty((b, t, spec.inner), dtype=proj.dtype, device=proj.device)
-    a.v = v.data_ptr()
+    y = torch.empty((b, t, spec.inner), dtype=proj.dtype, device=proj.device)
+    a.y = y.data_ptr()
     stream = cuda_ops._stream()  # pylint: disable=protected-access
     check = cuda_ops._check  # pylint: disable=protected-access
     if decode:

@@ -59,7 +59,8 @@ def _args():
     ap.add_argument("--kernel_table", default=None, help="after the timed regions, profile two more steps with the "
                     "torch profiler and write per-kernel device-time shares to this file (rank 0)")
     ap.add_argument("--serving", action="store_true", help="non-headline: prefill and decode throughput of the Sagisun "
-                    "design beside the Fuji decoder of equal widths, one JSON line per (size, model, batch)")
+                    "and Zukitar designs beside the Fuji decoder of equal widths, one JSON line per (size, model, batch)")
+    ap.add_argument("--serving_models", default=None, help="--serving: comma-separated subset of the models")
     ap.add_argument("--serving_sizes", default=None, help="--serving: comma-separated subset of the sizes")
     ap.add_argument("--serving_table", default=None, help="--serving: write per-kernel device times to this file")
     ap.add_argument("--skip_parity", action="store_true", help="N>1: skip the one-step fused-vs-library parity record")
@@ -140,6 +141,7 @@ def main():
         sampler.start()
         bench_serving.run(steps=args.steps, warmup=args.warmup, table=args.serving_table,
                           sizes=args.serving_sizes.split(",") if args.serving_sizes else None,
+                          models=args.serving_models.split(",") if args.serving_models else None,
                           emit=lambda line: print(line, flush=True))
         print(json.dumps({"clocks": sampler.stop()}))
         return
