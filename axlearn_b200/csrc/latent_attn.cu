@@ -10,7 +10,8 @@
 // valid (null: T).
 //
 //   latent_prep_kernel    norm of the latent, rotation of the key part, cache row; rotation of the queries
-//                         (in place, or into the rows that latent attention reads).
+//                         (in place, or into the rows that latent attention reads); latent_prep_vec_kernel is
+//                         its form for aligned bf16 prompts.
 //   latent_decode_kernel  bf16: 16 or 32 heads of one query token per CTA on the tensor cores, the cached rows
 //                         streamed once through shared memory; long caches are split over CTAs and
 //                         latent_merge_kernel joins the parts.
@@ -131,6 +132,92 @@ __global__ void __launch_bounds__(kLpThreads) latent_prep_kernel(LatentArgs a, i
       x[1] = T(v * cs.x + u * cs.y);
     }
   }
+}
+
+// Prompts with 16-byte aligned parts: four tokens per CTA, one warp each for the latent and one for the queries,
+// which are rotated in place.
+constexpr int kLvTokens = 4;
+
+__global__ void __launch_bounds__(64 * kLvTokens) latent_prep_vec_kernel(LatentArgs a) {
+  using bf16 = __nv_bfloat16;
+  extern __shared__ float2 s_turn[];  // [4][rot_dims / 2] (cos, sin)
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = a.rot_dims / 2;
+  const int64_t tokens = static_cast<int64_t>(a.B) * a.T, first = static_cast<int64_t>(blockIdx.x) * kLvTokens;
+  for (int i = tid; i < kLvTokens * half; i += 64 * kLvTokens) {
+    const int64_t row = min(first + i / half, tokens - 1);
+    const int pos = token_position(a, static_cast<int>(row / a.T), static_cast<int>(row % a.T));
+    const double turn = 6.283185307179586476925286766559;
+    double angle = max(pos, 0) * a.freq[i % half];
+    angle -= turn * rint(angle * (1.0 / turn));
+    float s, c;
+    sincosf(static_cast<float>(angle), &s, &c);
+    s_turn[i] = make_float2(c, s);
+  }
+  const int64_t row = first + warp % kLvTokens;
+  const float2* cs = s_turn + (warp % kLvTokens) * half;
+  const bool valid = row < tokens;
+  bf16* src = static_cast<bf16*>(const_cast<void*>(a.proj)) + (valid ? row : 0) * a.ld;
+  // Eight consecutive elements from element c on of a rotated part.
+  auto turn8 = [&](const uint4& u, int c) {
+    const uint32_t in[4] = {u.x, u.y, u.z, u.w};
+    uint32_t o[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 x = unpack2(in[i]);
+      const float2 t = c + 2 * i < a.rot_dims ? cs[(c >> 1) + i] : make_float2(1.f, 0.f);
+      o[i] = pack2(x.x * t.x - x.y * t.y, x.y * t.x + x.x * t.y);
+    }
+    return make_uint4(o[0], o[1], o[2], o[3]);
+  };
+  if (warp >= kLvTokens) {
+    const int head_w = a.dim + a.rot_dim, per = a.rot_dim / 8, items = a.heads * per;
+    bf16* q = src + a.q_off + a.dim;
+    __syncthreads();
+    if (!valid) return;
+#pragma unroll 4
+    for (int i = lane; i < items; i += 32) {
+      const int c = i % per * 8;
+      uint4* x = reinterpret_cast<uint4*>(q + static_cast<int64_t>(i / per) * head_w + c);
+      *x = turn8(*x, c);
+    }
+    return;
+  }
+  const int b = static_cast<int>((valid ? row : 0) / a.T), t = static_cast<int>((valid ? row : 0) % a.T);
+  const int pos = token_position(a, b, t);
+  float sq = 0.f;
+  for (int c = lane * 8; c < a.rank; c += 256) {
+    const uint4 u = *reinterpret_cast<const uint4*>(src + a.c_off + c);
+    const uint32_t in[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 x = unpack2(in[i]);
+      sq += x.x * x.x + x.y * x.y;
+    }
+  }
+  for (int off = 16; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
+  const float inv = 1.f / sqrtf(sq / a.rank + a.eps);
+  __syncthreads();
+  if (!valid) return;
+  bf16* dst = pos >= 0 ? static_cast<bf16*>(a.cache) + (static_cast<int64_t>(b) * a.slots + pos) * a.cache_ld : nullptr;
+  bf16* lat = static_cast<bf16*>(a.lat) + row * a.lat_ld;
+  for (int c = lane * 8; c < a.rank; c += 256) {
+    const uint4 u = *reinterpret_cast<const uint4*>(src + a.c_off + c);
+    const uint32_t in[4] = {u.x, u.y, u.z, u.w};
+    const float4 w0 = *reinterpret_cast<const float4*>(a.norm_w + c), w1 = *reinterpret_cast<const float4*>(a.norm_w + c + 4);
+    const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+    uint32_t o[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 x = unpack2(in[i]);
+      o[i] = pack2(x.x * inv * w[2 * i], x.y * inv * w[2 * i + 1]);
+    }
+    const uint4 y = make_uint4(o[0], o[1], o[2], o[3]);
+    if (dst != nullptr) *reinterpret_cast<uint4*>(dst + c) = y;
+    *reinterpret_cast<uint4*>(lat + c) = y;
+  }
+  if (dst != nullptr)
+    for (int c = lane * 8; c < a.rot_dim; c += 256)
+      *reinterpret_cast<uint4*>(dst + a.rot_off + c) = turn8(*reinterpret_cast<const uint4*>(src + a.r_off + c), c);
 }
 
 constexpr int kLaThreads = 256, kLaKeys = 64, kLaCols = 8;
@@ -502,6 +589,14 @@ extern "C" int axb_latent_prep(const axb::LatentArgs* args, cudaStream_t stream)
   if (axb::latent_bad(a)) return -10;
   const size_t smem = sizeof(float2) * (a.rot_dims / 2);
   if (smem > 48 * 1024) return -10;
+  const int aligned = a.ld | a.cache_ld | a.lat_ld | a.dim | a.rot_dim | a.rank | a.q_off | a.c_off | a.r_off;
+  if (a.act_bf16 && a.qbuf == nullptr && a.lat != nullptr && !(aligned & 7)) {
+    const int64_t ctas = (static_cast<int64_t>(a.B) * a.T + axb::kLvTokens - 1) / axb::kLvTokens;
+    if (smem * axb::kLvTokens <= 48 * 1024) {
+      axb::latent_prep_vec_kernel<<<static_cast<unsigned>(ctas), 64 * axb::kLvTokens, smem * axb::kLvTokens, stream>>>(a);
+      return axb::latent_launched();
+    }
+  }
   // Few tokens: the heads side by side; many: fewer copies of the trigonometry.
   const int heads_per = static_cast<int64_t>(a.B) * a.T <= 1024 ? 4 : 32;
   const dim3 grid(a.T, a.B, 1 + (a.heads + heads_per - 1) / heads_per);

@@ -13,6 +13,7 @@ import collections
 import functools
 import gc
 import json
+import statistics
 from typing import Optional
 
 import torch
@@ -48,14 +49,16 @@ def _fuji_engine(size: str, layers: int, batch: int, max_len: int) -> DecodeEngi
 
 
 def _time(fn, repeat: int) -> float:
-    start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    """Median device time of a call in ms (an allocation that grows the memory pool takes as long as several
+    passes and would swamp a mean)."""
+    events = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(repeat)]
     torch.cuda.synchronize()
-    start.record()
-    for _ in range(repeat):
+    for start, end in events:
+        start.record()
         fn()
-    end.record()
+        end.record()
     torch.cuda.synchronize()
-    return start.elapsed_time(end) / repeat
+    return statistics.median(start.elapsed_time(end) for start, end in events)
 
 
 def _kernel_times(fn) -> list:
