@@ -189,7 +189,7 @@ def padded_group_layout(expert_of_pair: torch.Tensor, num_experts: int, max_rows
 
 
 def _grouped_argtypes():
-    h = _lib()
+    h = cuda_ops.lib()      # not _lib(): a process may have the products without the dispatch kernels
     if not getattr(h, "_axb_grouped_configured", False):
         h.axb_gemm_bf16_grouped.argtypes = [
             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int, c_int, c_int,
