@@ -52,7 +52,7 @@ def _latent_spec(heads, dim, rot, vdim, rank, rot_dims=None):
                                  1.3 * (dim + rot) ** -0.5, 1e-5)
 
 
-LATENT_SIZES = [(4, 64, 16, 64, 128), (16, 128, 64, 128, 512), (5, 40, 24, 72, 96), (33, 32, 8, 16, 264), (3, 7, 6, 5, 11),
+LATENT_SIZES = [(6, 64, 32, 48, 160), (16, 128, 64, 128, 512), (5, 40, 24, 72, 96), (33, 32, 8, 16, 264), (3, 7, 6, 5, 11),
                 (2, 8, 8, 128, 8), (40, 128, 64, 64, 504), (2, 128, 64, 192, 640)]
 
 
@@ -106,18 +106,18 @@ def test_latent_step(sizes, t, dtype, form):
 @pytest.mark.parametrize("far", [0, 63, 64, 127, 128, 130, 191, 192, 639])
 def test_one_cached_row_stands_out(far):
     """A key that outweighs hundreds of others, at the edges of tiles and splits: the output is its value."""
-    spec = _latent_spec(8, 64, 16, 64, 128)
+    spec = _latent_spec(8, 48, 24, 64, 192)
     proj, norm, uk, uv, cols = _latent_case(spec, 1, 1, BF16, seed=3)
     rows = torch.zeros(1, 640, spec.row_width, device="cuda", dtype=BF16)
-    rows[..., :128] = _randn(1, 640, 128, seed=4, dtype=BF16)
-    q = proj[0, 0, :8 * 80].reshape(8, 80).float()
-    lat = torch.einsum("hd,rhd->hr", q[:, :64], uk[:, :512].float().reshape(128, 8, 64))
-    rows[0, far, :128] = (lat[5] * 40 / lat[5].norm()).to(BF16)        # head 5 points there
+    rows[..., :192] = _randn(1, 640, 192, seed=4, dtype=BF16)
+    q = proj[0, 0, :8 * 72].reshape(8, 72).float()
+    lat = torch.einsum("hd,rhd->hr", q[:, :48], uk[:, :8 * 48].float().reshape(192, 8, 48))
+    rows[0, far, :192] = (lat[5] * 40 / lat[5].norm()).to(BF16)        # head 5 points there
     start = _ints(639)
     with use_reference_ops():
         want, _ = latent_ops.latent_attention(proj, norm, uk, uv, spec, cols, start=start, cache={"latent": rows.clone()})
     got, _ = latent_ops.latent_attention(proj.clone(), norm, uk, uv, spec, cols, start=start, cache={"latent": rows.clone()})
-    value = (uv[:512].float() @ rows[0, far, :128].float()).reshape(8, 64)[5]
+    value = (uv[:512].float() @ rows[0, far, :192].float()).reshape(8, 64)[5]
     if far != 639:      # the new token's own row is written by the step
         assert _rel(want[0, 0].reshape(8, 64)[5], value) < 0.05
     assert _rel(got, want) < 0.015
@@ -155,7 +155,7 @@ def _copy(state):
     return {k: v.clone() for k, v in state.items()}
 
 
-SSD_SIZES = [(8, 64, 128, 1, 4, 1), (6, 48, 48, 2, 3, 3), (4, 16, 24, 4, 2, 2), (2, 128, 64, 1, 4, 1), (3, 5, 7, 3, 5, 3),
+SSD_SIZES = [(8, 64, 128, 1, 4, 1), (6, 40, 56, 2, 3, 3), (4, 16, 24, 4, 2, 2), (2, 128, 64, 1, 4, 1), (3, 5, 7, 3, 5, 3),
              (3, 80, 128, 1, 4, 2), (2, 200, 16, 2, 1, 1), (2, 32, 200, 1, 4, 1)]
 
 
@@ -241,7 +241,7 @@ def test_ssd_chunk_keeps_small_differences():
 
 
 # ------------------------------------------------------------------------------ experts
-EXPERT_SIZES = [(16, 1, 256, 96, 1.0), (32, 4, 512, 320, 7.0), (5, 5, 40, 24, 0.6), (300, 8, 64, 64, 2.0), (1, 1, 72, 8, 1.0),
+EXPERT_SIZES = [(12, 1, 320, 72, 0.8), (32, 4, 512, 320, 7.0), (5, 5, 40, 24, 0.6), (300, 8, 64, 64, 2.0), (1, 1, 72, 8, 1.0),
                 (7, 2, 42, 13, 1.5)]
 
 
